@@ -14,6 +14,7 @@ from .tufirax_config import TufiraxConfig
 from .vipelix_config import VipelixConfig
 from .tibepel_config import TibepelConfig
 from .tugodra_config import TugodraConfig
+from .sozudra_config import SozudraConfig
 
 _ARCHITECTURES: Dict[str, Type] = {}
 
@@ -59,3 +60,4 @@ register_architecture("Tufirax", TufiraxConfig)
 register_architecture("Vipelix", VipelixConfig)
 register_architecture("Tibepel", TibepelConfig)
 register_architecture("Tugodra", TugodraConfig)
+register_architecture("Sozudra", SozudraConfig)

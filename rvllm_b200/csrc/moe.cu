@@ -8,9 +8,10 @@
 //
 //   moe_route_top act on a router's float32 logits: s = sigmoid(z); the choice is made among s + correction, within the best
 //                 `keep` of `groups` equal groups of neighbouring experts (a group counts by the sum of its two largest
-//                 corrected scores); chosen [tokens, top], weights = the chosen s over their sum (+ eps)
+//                 corrected scores); chosen [tokens, top], weights = the chosen s over their sum (+ eps).  With `softmax`
+//                 the choice is made among z + correction itself and the weights are the softmax over the chosen ones
 //   moe_gate_up   act[t * top + k, f] = silu(gate_e[f] . x_t) * (up_e[f] . x_t)  or  relu(up_e[f] . x_t)^2,  e = chosen[t, k]
-//   moe_down      out[t, n] = (add[t, n]) + weight * sum_k weights[t, k] down_e(k)[n] . act[t * top + k]
+//   moe_down      out[t, n] = (add_scale[t] add[t, n]) + weight * sum_k weights[t, k] down_e(k)[n] . act[t * top + k]
 //
 // One CTA per (token, slot) and block of features keeps the token's vector in shared memory as float; a warp owns a
 // feature at a time and its lanes walk the weight row (16-byte loads where rows are aligned).  The weights of an
@@ -24,7 +25,7 @@
 //   moe_route     row_of[pair], src_of[row] and the products' work units (tile_group, tile_rows) from chosen (one CTA:
 //                 counts, padded offsets, places)
 //   moe_gather    xs[row] = x[src_of[row]], zeros in the padding
-//   moe_combine   out[t] = (add[t]) + weight * sum_k weights[t, k] ys[row_of[t * top + k]]   (slots in their order: one sum per element)
+//   moe_combine   out[t] = (add_scale[t] add[t]) + weight * sum_k weights[t, k] ys[row_of[t * top + k]]   (slots in their order: one sum per element)
 #include "common.cuh"
 
 // N rows of W against one vector at a time: the lanes walk all rows together, so N loads are in flight per lane and step
@@ -132,7 +133,8 @@ moe_gate_up_kernel(const T* __restrict__ x, const int* __restrict__ chosen, cons
 template <typename T, typename TO>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
 moe_down_kernel(const T* __restrict__ act, const int* __restrict__ chosen, const T* __restrict__ down, const float* add,
-                TO* out, int top, int experts, int ff, int width, float weight, const float* __restrict__ weights) {
+                TO* out, int top, int experts, int ff, int width, float weight, const float* __restrict__ weights,
+                const float* __restrict__ add_scale) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     extern __shared__ float as[];                 // [top][ff]
@@ -161,7 +163,7 @@ moe_down_kernel(const T* __restrict__ act, const int* __restrict__ chosen, const
         const int n = n0 + warp + j * MOE_WARPS;
         if (lane == 0 && n < width) {
             float v = sum[j] * weight;
-            if (add) v += add[(size_t)t * width + n];
+            if (add) v += add_scale ? add_scale[t] * add[(size_t)t * width + n] : add[(size_t)t * width + n];
             out[(size_t)t * width + n] = rv_from_float<TO>(v);
         }
     }
@@ -171,8 +173,8 @@ static RvPerDevice g_once[8];
 
 template <typename T>
 static int moe_launch(const void* x, const int* chosen, const float* weights, const void* gate_up, const void* down, void* act,
-                      const float* add, void* out, int out_f32, int tokens, int top, int experts, int ff, int width, float weight,
-                      int gated, int slot, cudaStream_t stream) {
+                      const float* add, const float* add_scale, void* out, int out_f32, int tokens, int top, int experts, int ff,
+                      int width, float weight, int gated, int slot, cudaStream_t stream) {
     const int smem_a = width * 4, smem_b = top * ff * 4;
     if (smem_a > 200 * 1024 || smem_b > 200 * 1024) return RV_ERR_UNSUPPORTED;
     int st;
@@ -195,38 +197,39 @@ static int moe_launch(const void* x, const int* chosen, const float* weights, co
         st = rv_configure_smem(g_once[slot + 1], moe_down_kernel<T, float>, 200 * 1024);
         if (st != RV_OK) return st;
         RV_LAUNCH_ST = rv_launch(moe_down_kernel<T, float>, dim3(grid), dim3(MOE_WARPS * 32), (size_t)smem_b, stream, (const T*)act,
-                                 chosen, (const T*)down, add, (float*)out, top, experts, ff, width, weight, weights);
+                                 chosen, (const T*)down, add, (float*)out, top, experts, ff, width, weight, weights, add_scale);
     } else {
         st = rv_configure_smem(g_once[slot + 2], moe_down_kernel<T, T>, 200 * 1024);
         if (st != RV_OK) return st;
         RV_LAUNCH_ST = rv_launch(moe_down_kernel<T, T>, dim3(grid), dim3(MOE_WARPS * 32), (size_t)smem_b, stream, (const T*)act,
-                                 chosen, (const T*)down, add, (T*)out, top, experts, ff, width, weight, weights);
+                                 chosen, (const T*)down, add, (T*)out, top, experts, ff, width, weight, weights, add_scale);
     }
     return rv_launch_status();
 }
 
-// x [tokens, width], act [tokens * top, ff] (scratch of the weights' type), add float [tokens, width] or null,
+// x [tokens, width], act [tokens * top, ff] (scratch of the weights' type), add float [tokens, width] or null, add_scale float
+// [tokens] or null (1),
 // weights float [tokens, top] or null, out [tokens, width] float (out_f32) or of the weights' type.  gated: 1 the experts'
 // first matrix is [gate | up] with SiLU, 0 it is the up matrix with a squared relu.  Two launches.
 RV_EXPORT int rv_moe_experts_ex(const void* x, const int* chosen, const float* weights, const void* gate_up, const void* down, void* act,
-                                const float* add, void* out, int out_f32, int tokens, int top, int experts, int ff, int width,
-                                float weight, int gated, int dtype, cudaStream_t stream) {
+                                const float* add, const float* add_scale, void* out, int out_f32, int tokens, int top, int experts,
+                                int ff, int width, float weight, int gated, int dtype, cudaStream_t stream) {
     if (tokens < 0 || top <= 0 || experts <= 0 || ff <= 0 || width <= 0) return RV_ERR_BAD_SIZE;
     if ((long long)tokens * top > 0x7fffffffLL || ff > 65535 * MOE_FEATURES || width > 65535 * MOE_FEATURES) return RV_ERR_BAD_SIZE;
     if (tokens == 0) return RV_OK;
     if (dtype == RV_DTYPE_F32)
-        return moe_launch<float>(x, chosen, weights, gate_up, down, act, add, out, 1, tokens, top, experts, ff, width, weight, gated, 0, stream);
+        return moe_launch<float>(x, chosen, weights, gate_up, down, act, add, add_scale, out, 1, tokens, top, experts, ff, width, weight, gated, 0, stream);
     if (dtype == RV_DTYPE_BF16)
-        return moe_launch<__nv_bfloat16>(x, chosen, weights, gate_up, down, act, add, out, out_f32, tokens, top, experts, ff, width, weight,
-                                         gated, 4, stream);
+        return moe_launch<__nv_bfloat16>(x, chosen, weights, gate_up, down, act, add, add_scale, out, out_f32, tokens, top, experts, ff, width,
+                                         weight, gated, 4, stream);
     return RV_ERR_BAD_DTYPE;
 }
 
 RV_EXPORT int rv_moe_experts(const void* x, const int* chosen, const void* gate_up, const void* down, void* act, const float* add,
                              void* out, int out_f32, int tokens, int top, int experts, int ff, int width, float weight,
                              int dtype, cudaStream_t stream) {
-    return rv_moe_experts_ex(x, chosen, nullptr, gate_up, down, act, add, out, out_f32, tokens, top, experts, ff, width, weight, 1, dtype,
-                             stream);
+    return rv_moe_experts_ex(x, chosen, nullptr, gate_up, down, act, add, nullptr, out, out_f32, tokens, top, experts, ff, width, weight, 1,
+                             dtype, stream);
 }
 
 // ------------------------------------------------------------------ sorting pairs by expert for the grouped products
@@ -306,7 +309,8 @@ __global__ void moe_gather_kernel(const uint4* __restrict__ x, const int* __rest
 
 template <typename TO>
 __global__ void moe_combine_kernel(const float* __restrict__ ys, const int* __restrict__ row_of, const float* add, TO* out,
-                                   int top, int width, float weight, size_t total, const float* __restrict__ weights) {
+                                   int top, int width, float weight, size_t total, const float* __restrict__ weights,
+                                   const float* __restrict__ add_scale) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
@@ -318,7 +322,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ ys, const int* __re
             if (row >= 0) s = fmaf(weights ? weights[t * top + k] : 1.f, ys[(size_t)row * width + n], s);
         }
         float v = s * weight;
-        if (add) v += add[i];
+        if (add) v += add_scale ? add_scale[t] * add[i] : add[i];
         out[i] = rv_from_float<TO>(v);
     }
 }
@@ -346,16 +350,16 @@ RV_EXPORT int rv_moe_gather(const void* x, const int* src_of, void* xs, int rows
 }
 
 RV_EXPORT int rv_moe_combine(const float* ys, const int* row_of, const float* add, void* out, int out_f32, int tokens, int top,
-                             int width, float weight, const float* weights, cudaStream_t stream) {
+                             int width, float weight, const float* weights, const float* add_scale, cudaStream_t stream) {
     if (tokens < 0 || top <= 0 || width <= 0) return RV_ERR_BAD_SIZE;
     if (tokens == 0) return RV_OK;
     const size_t total = (size_t)tokens * width;
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     if (out_f32)
-        RV_LAUNCH_ST = rv_launch(moe_combine_kernel<float>, dim3(blocks), dim3(256), 0, stream, ys, row_of, add, (float*)out, top, width, weight, total, weights);
+        RV_LAUNCH_ST = rv_launch(moe_combine_kernel<float>, dim3(blocks), dim3(256), 0, stream, ys, row_of, add, (float*)out, top, width, weight, total, weights, add_scale);
     else
         RV_LAUNCH_ST = rv_launch(moe_combine_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, ys, row_of, add, (__nv_bfloat16*)out, top,
-                                 width, weight, total, weights);
+                                 width, weight, total, weights, add_scale);
     return rv_launch_status();
 }
 
@@ -380,7 +384,7 @@ __device__ __forceinline__ void mr_argmax(const float* v, int n, int lane, float
 __global__ void __launch_bounds__(MR_WARPS * 32)
 moe_route_top_kernel(const float* __restrict__ logits, int stride, const float* __restrict__ correction, int* __restrict__ chosen,
                      float* __restrict__ weights, float* __restrict__ gate_out, int tokens, int experts, int top, int groups, int keep,
-                     float weight_eps) {
+                     float weight_eps, int softmax) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     extern __shared__ float mr_smem[];
@@ -392,9 +396,9 @@ moe_route_top_kernel(const float* __restrict__ logits, int stride, const float* 
     float* gs = c + experts;
     const float* z = logits + (size_t)t * stride;
     for (int e = lane; e < experts; e += 32) {
-        const float v = 1.0f / (1.0f + expf(-z[e]));
+        const float v = softmax ? z[e] + correction[e] : 1.0f / (1.0f + expf(-z[e]));
         s[e] = v;
-        c[e] = v + correction[e];
+        c[e] = softmax ? v : v + correction[e];
     }
     if (gate_out && lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-z[experts]));
     __syncwarp();
@@ -419,12 +423,13 @@ moe_route_top_kernel(const float* __restrict__ logits, int stride, const float* 
             if (gs[e / per] != -INFINITY) c[e] = -INFINITY;  // (a kept group was set to -inf when it was taken)
         __syncwarp();
     }
-    float sum = 0.f, mine = 0.f;
+    float sum = 0.f, mine = 0.f, largest = 0.f;
     for (int k = 0; k < top; ++k) {
         float best; int at;
         mr_argmax(c, experts, lane, best, at);
         if (at >= experts) at = 0;                           // (cannot happen: top <= the experts of the kept groups)
-        const float w = s[at];
+        if (k == 0) largest = s[at];                         // (with one score per expert the first choice has the largest)
+        const float w = softmax ? expf(s[at] - largest) : s[at];
         sum += w;
         if (lane == k % 32 && k < 32) mine = w;
         if (lane == 0) {
@@ -442,7 +447,7 @@ moe_route_top_kernel(const float* __restrict__ logits, int stride, const float* 
 
 // logits float [tokens, stride]: the experts' logits and, with gate_out, one more column whose sigmoid goes to gate_out.
 RV_EXPORT int rv_moe_route_top(const float* logits, int stride, const float* correction, int* chosen, float* weights, float* gate_out,
-                               int tokens, int experts, int top, int groups, int keep, float weight_eps, cudaStream_t stream) {
+                               int tokens, int experts, int top, int groups, int keep, float weight_eps, int softmax, cudaStream_t stream) {
     if (tokens < 0 || experts <= 0 || top <= 0 || top > experts || groups <= 0 || experts % groups || keep <= 0 || keep > groups)
         return RV_ERR_BAD_SIZE;
     if (stride < experts + (gate_out ? 1 : 0) || top > (experts / groups) * keep) return RV_ERR_BAD_SIZE;
@@ -450,6 +455,6 @@ RV_EXPORT int rv_moe_route_top(const float* logits, int stride, const float* cor
     if (tokens == 0) return RV_OK;
     const size_t smem = (size_t)MR_WARPS * (2 * experts + groups) * sizeof(float);
     RV_LAUNCH_ST = rv_launch(moe_route_top_kernel, dim3((tokens + MR_WARPS - 1) / MR_WARPS), dim3(MR_WARPS * 32), smem, stream, logits,
-                             stride, correction, chosen, weights, gate_out, tokens, experts, top, groups, keep, weight_eps);
+                             stride, correction, chosen, weights, gate_out, tokens, experts, top, groups, keep, weight_eps, softmax);
     return rv_launch_status();
 }

@@ -1,123 +1,298 @@
-// What stands between the stacked q/k/v product and the attention kernels for mixers whose queries and keys are
-// rotated and then made unit-RMS vectors per head:
+// What stands around the attention kernels for mixers whose queries and keys are rotated and then, optionally, made
+// unit-RMS vectors per head, whose heads may carry two maps, and whose values may turn with their position:
 //
-//   qk_unit_prepare   rows [q: nh x d | k: nkv x d | v: nkv x vd | gate logits: nh] of a float32 projection (k and v only
-//                     where the layer has them).  The leading `rot` elements of every head of q and k turn by the angle
-//                     of (position, pair): pairs (2i, 2i + 1), or (i, i + rot / 2) with `halves`; then the head is divided
-//                     by sqrt(mean(x^2) + eps) over its d elements (no weight).  q goes to q_out [T, nh, P], k and v
-//                     into the token's cache slot (planes 0 and 1 of [pages, 2, nkv, page, P]); P >= max(d, vd), and
-//                     what lies beyond a head's d (or vd) elements is written as zeros.  sigmoid of the gate logits
-//                     goes to a float array.  A token with slot -1 writes no key and no value.
+//   qk_prepare        rows [q: nh x M x d | k: nkv x M x d | v: nkv x vd | gate logits: nh] of a float32 projection (k and v
+//                     only where the layer has them; M = 1 or 2 maps per head), plus a bias per column (optional).  The
+//                     leading `rot` elements of every map of q and k turn by the angle of (position, pair): pairs
+//                     (2i, 2i + 1), or (i, i + rot / 2) with `halves`; with `unit` the map is then divided by
+//                     sqrt(mean(x^2) + eps) over its d elements (no weight).  With value tables the value turns too, over all
+//                     its vd elements in the same layout of pairs.  q goes to q_out [T, nh, M, P], k and v into the token's
+//                     cache slot (planes 0 and 1 of [pages, 2, nkv, page, P]); P >= max(M d, vd).  A query row of map m holds
+//                     its d elements at m d, a key row all maps side by side, so that (query row of map m) . (key row) is
+//                     map m's score; everything else of a row is written as zeros.  sigmoid of the gate logits goes to a
+//                     float array.  A token with slot -1 writes no key and no value.
+//   turn_back         rows of attention results [T, nh, P]: the leading vd elements of every head turned by MINUS the token's
+//                     angle, written as [T, nh, vd]
+//   map_difference    rows [T, nh, 2, P] of two maps' results: o = a1 - lambda a2 over the leading vd elements, then
+//                     o / sqrt(mean(o^2) + eps) * factor, written as [T, nh, vd]
 //
 // All arithmetic is float; the results are rounded once, when they are stored (float or bfloat16).
 #include "common.cuh"
 
 #define QP_WARPS 8
-#define QP_MAX_DIM 256
+#define QP_MAX_DIM 1024
 
 __device__ __forceinline__ void qp_store(void* p, int dtype, size_t i, float v) {
     if (dtype == RV_DTYPE_F32) ((float*)p)[i] = v;
     else ((__nv_bfloat16*)p)[i] = __float2bfloat16_rn(v);
 }
 
-// One block per token; a warp takes one head of q, k or v at a time.  NJ: elements of a head slot per lane (P <= 32 NJ).
+struct QkPrepareArgs {
+    const float* proj; int row_stride;
+    const float* bias;                                          // one per column of q, k and v, or null
+    const int* positions; const float *cos_t, *sin_t; int rot, table_rows, halves;
+    const float *vcos_t, *vsin_t; int v_table_rows;            // value tables [rows, vd / 2] or null
+    const int* slot_mapping; void *cache, *q_out; int out_dtype; float* gate_out;
+    int nh, nkv, d, vd, P, maps, page_size; float eps; int unit, write_kv;
+};
+
+// Element e of a vector of which the leading `rot` elements turn; `cs` and `sn` are the token's rows of the tables.
+__device__ __forceinline__ float qp_turned(const float* v, int e, int rot, int halves, const float* __restrict__ cs,
+                                           const float* __restrict__ sn) {
+    const float x = v[e];
+    if (e >= rot) return x;
+    if (halves) {
+        const int half = rot >> 1;
+        const bool first = e < half;
+        const int p = first ? e : e - half;
+        const float other = v[first ? e + half : e - half];
+        return first ? x * cs[p] - other * sn[p] : x * cs[p] + other * sn[p];
+    }
+    const int p = e >> 1;
+    const float other = v[e ^ 1];
+    return (e & 1) ? x * cs[p] + other * sn[p] : x * cs[p] - other * sn[p];
+}
+
+// One block per token; a warp takes one map of a head of q or k, or one head of v, at a time.  NJ: elements of a head slot
+// per lane (P <= 32 NJ).
 template <int NJ>
 __global__ void __launch_bounds__(QP_WARPS * 32)
-qk_unit_prepare_kernel(const float* __restrict__ proj, int row_stride, const int* __restrict__ positions,
-                       const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot, int table_rows, int halves,
-                       const int* __restrict__ slot_mapping, void* __restrict__ cache, void* __restrict__ q_out, int out_dtype,
-                       float* __restrict__ gate_out, int nh, int nkv, int d, int vd, int P, int page_size, float eps, int write_kv) {
+qk_prepare_kernel(const QkPrepareArgs a) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     __shared__ float buf[QP_WARPS][32 * NJ];
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const size_t row = (size_t)t * row_stride;
-    int pos = positions[t];
+    const size_t row = (size_t)t * a.row_stride;
+    int pos = a.positions[t];
     if (pos < 0) pos = 0;
-    if (pos >= table_rows) pos = table_rows - 1;      // the host refuses such positions; never read outside
-    const int half = rot >> 1;
-    const float* cs = cos_t ? cos_t + (size_t)pos * half : nullptr;
-    const float* sn = sin_t ? sin_t + (size_t)pos * half : nullptr;
-    const int slot = write_kv ? slot_mapping[t] : -1;
-    const int items = nh + (write_kv ? 2 * nkv : 0);
+    const int qk_pos = pos < a.table_rows ? pos : a.table_rows - 1;      // the host refuses such positions; never read outside
+    const int v_pos = pos < a.v_table_rows ? pos : a.v_table_rows - 1;
+    const float* cs = a.cos_t ? a.cos_t + (size_t)qk_pos * (a.rot >> 1) : nullptr;
+    const float* sn = a.sin_t ? a.sin_t + (size_t)qk_pos * (a.rot >> 1) : nullptr;
+    const float* vcs = a.vcos_t ? a.vcos_t + (size_t)v_pos * (a.vd >> 1) : nullptr;
+    const float* vsn = a.vcos_t ? a.vsin_t + (size_t)v_pos * (a.vd >> 1) : nullptr;
+    const int slot = a.write_kv ? a.slot_mapping[t] : -1;
+    const int nq = a.nh * a.maps, nk = a.nkv * a.maps;
+    const int items = nq + (a.write_kv ? nk + a.nkv : 0);
     float* mine = buf[warp];
     for (int item = warp; item < items; item += QP_WARPS) {
-        const int kind = item < nh ? 0 : (item < nh + nkv ? 1 : 2);          // q, k, v
-        const int head = kind == 0 ? item : (kind == 1 ? item - nh : item - nh - nkv);
+        const int kind = item < nq ? 0 : (item < nq + nk ? 1 : 2);            // q, k, v
+        const int index = kind == 0 ? item : (kind == 1 ? item - nq : item - nq - nk);
         if (kind != 0 && slot < 0) continue;                                  // (the same for the whole warp)
-        const int n = kind == 2 ? vd : d;
-        const size_t src = row + (kind == 0 ? (size_t)head * d
-                                            : (kind == 1 ? (size_t)nh * d + (size_t)head * d
-                                                         : (size_t)(nh + nkv) * d + (size_t)head * vd));
-        for (int i = lane; i < n; i += 32) mine[i] = proj[src + i];
+        const int n = kind == 2 ? a.vd : a.d;
+        const int head = kind == 2 ? index : index / a.maps, map = kind == 2 ? 0 : index - head * a.maps;
+        const size_t col = kind == 0 ? (size_t)index * a.d
+                                     : (kind == 1 ? (size_t)(nq + index) * a.d : (size_t)(nq + nk) * a.d + (size_t)index * a.vd);
+        for (int i = lane; i < n; i += 32) mine[i] = a.proj[row + col + i] + (a.bias ? a.bias[col + i] : 0.f);
         __syncwarp();
+        const float* c = kind == 2 ? vcs : cs;
+        const float* s = kind == 2 ? vsn : sn;
+        const int rot = c ? (kind == 2 ? a.vd : a.rot) : 0;
+        const int at = map * a.d;                                             // where the map lies in its row
         float vals[NJ];
         float ss = 0.f;
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
-            const int i = lane + 32 * j;
-            float v = i < n ? mine[i] : 0.f;
-            if (kind != 2 && i < rot) {
-                if (halves) {
-                    const bool first = i < half;
-                    const int p = first ? i : i - half;
-                    const float other = mine[first ? i + half : i - half];
-                    v = first ? v * cs[p] - other * sn[p] : v * cs[p] + other * sn[p];
-                } else {
-                    const int p = i >> 1;
-                    const float other = mine[i ^ 1];
-                    v = (i & 1) ? v * cs[p] + other * sn[p] : v * cs[p] - other * sn[p];
-                }
-            }
+            const int e = lane + 32 * j - at;
+            const float v = (e >= 0 && e < n) ? qp_turned(mine, e, rot, a.halves, c, s) : 0.f;
             vals[j] = v;
             ss = fmaf(v, v, ss);
         }
         float r = 1.f;
-        if (kind != 2) {
+        if (kind != 2 && a.unit) {
             ss = rv_warp_sum(ss);
-            r = 1.0f / sqrtf(ss / (float)n + eps);
+            r = 1.0f / sqrtf(ss / (float)n + a.eps);
         }
         void* dst_base;
         size_t dst;
         if (kind == 0) {
-            dst_base = q_out;
-            dst = ((size_t)t * nh + head) * P;
+            dst_base = a.q_out;
+            dst = ((size_t)t * nq + index) * a.P;
         } else {
-            dst_base = cache;
-            const size_t page = (size_t)(slot / page_size), off = (size_t)(slot % page_size);
-            dst = (((page * 2 + (kind == 2 ? 1 : 0)) * nkv + head) * page_size + off) * P;
+            dst_base = a.cache;
+            const size_t page = (size_t)(slot / a.page_size), off = (size_t)(slot % a.page_size);
+            dst = (((page * 2 + (kind == 2 ? 1 : 0)) * a.nkv + head) * a.page_size + off) * a.P;
         }
+        // a key's maps are written by different warps: each its own elements, the last one the row's tail as well
+        const int lo = kind == 1 ? at : 0, hi = (kind == 1 && map + 1 < a.maps) ? at + a.d : a.P;
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
             const int i = lane + 32 * j;
-            if (i < P) qp_store(dst_base, out_dtype, dst + i, i < n ? vals[j] * r : 0.f);
+            if (i >= lo && i < hi) qp_store(dst_base, a.out_dtype, dst + i, vals[j] * r);
         }
         __syncwarp();
     }
-    if (gate_out) {
-        const size_t g0 = row + (size_t)nh * d + (write_kv ? (size_t)nkv * (d + vd) : 0);
-        for (int h = threadIdx.x; h < nh; h += blockDim.x)
-            gate_out[(size_t)t * nh + h] = 1.0f / (1.0f + expf(-proj[g0 + h]));
+    if (a.gate_out) {
+        const size_t g0 = row + (size_t)nq * a.d + (a.write_kv ? (size_t)nk * a.d + (size_t)a.nkv * a.vd : 0);
+        for (int h = threadIdx.x; h < a.nh; h += blockDim.x)
+            a.gate_out[(size_t)t * a.nh + h] = 1.0f / (1.0f + expf(-a.proj[g0 + h]));
     }
 }
 
-RV_EXPORT int rv_qk_unit_prepare(const float* proj, int row_stride, const int* positions, const float* cos_t, const float* sin_t,
-                                 int rot, int table_rows, int halves, const int* slot_mapping, void* cache, void* q_out, int out_dtype,
-                                 float* gate_out, int n_tokens, int nh, int nkv, int d, int vd, int P, int page_size, float eps,
-                                 int write_kv, cudaStream_t stream) {
-    if (n_tokens < 0 || nh <= 0 || nkv <= 0 || d <= 0 || vd <= 0 || P < d || P < vd || page_size <= 0 || table_rows <= 0)
+RV_EXPORT int rv_qk_prepare(const float* proj, int row_stride, const float* bias, const int* positions, const float* cos_t,
+                            const float* sin_t, int rot, int table_rows, int halves, const float* vcos_t, const float* vsin_t,
+                            int v_table_rows, const int* slot_mapping, void* cache, void* q_out, int out_dtype, float* gate_out,
+                            int n_tokens, int nh, int nkv, int d, int vd, int P, int maps, int page_size, float eps, int unit,
+                            int write_kv, cudaStream_t stream) {
+    if (n_tokens < 0 || nh <= 0 || nkv <= 0 || d <= 0 || vd <= 0 || P < vd || page_size <= 0 || table_rows <= 0 || v_table_rows <= 0)
         return RV_ERR_BAD_SIZE;
-    if (P > QP_MAX_DIM) return RV_ERR_UNSUPPORTED;
+    if (maps != 1 && maps != 2) return RV_ERR_BAD_SIZE;
+    if (P > QP_MAX_DIM || d > QP_MAX_DIM) return RV_ERR_UNSUPPORTED;
+    if (P < maps * d) return RV_ERR_BAD_SIZE;
     if (rot < 0 || rot > d || (rot & 1)) return RV_ERR_BAD_SIZE;
-    if (row_stride < nh * d + (write_kv ? nkv * (d + vd) : 0) + (gate_out ? nh : 0)) return RV_ERR_BAD_SIZE;
+    if ((vcos_t == nullptr) != (vsin_t == nullptr) || (vcos_t && (vd & 1))) return RV_ERR_BAD_SIZE;
+    if (row_stride < maps * nh * d + (write_kv ? nkv * (maps * d + vd) : 0) + (gate_out ? nh : 0)) return RV_ERR_BAD_SIZE;
     if (write_kv && (!slot_mapping || !cache)) return RV_ERR_BAD_SIZE;
     if (out_dtype & ~1) return RV_ERR_BAD_DTYPE;
     if (n_tokens == 0) return RV_OK;
-    if (!cos_t || !sin_t) rot = 0;
-    auto kernel = P <= 32 ? qk_unit_prepare_kernel<1> : (P <= 64 ? qk_unit_prepare_kernel<2> : (P <= 128 ? qk_unit_prepare_kernel<4>
-                                                                                                              : qk_unit_prepare_kernel<8>));
-    RV_LAUNCH_ST = rv_launch(kernel, dim3(n_tokens), dim3(QP_WARPS * 32), 0, stream, proj, row_stride, positions, cos_t,
-                             sin_t, rot, table_rows, halves, slot_mapping, cache, q_out, out_dtype, gate_out, nh, nkv, d, vd, P,
-                             page_size, eps, write_kv);
+    if (!cos_t || !sin_t) { cos_t = sin_t = nullptr; rot = 0; }
+    const QkPrepareArgs a = {proj, row_stride, bias, positions, cos_t, sin_t, rot, table_rows, halves, vcos_t, vsin_t, v_table_rows,
+                             slot_mapping, cache, q_out, out_dtype, gate_out, nh, nkv, d, vd, P, maps, page_size, eps, unit, write_kv};
+    auto kernel = P <= 32 ? qk_prepare_kernel<1> : (P <= 64 ? qk_prepare_kernel<2> : (P <= 128 ? qk_prepare_kernel<4>
+                : (P <= 256 ? qk_prepare_kernel<8> : qk_prepare_kernel<32>)));
+    RV_LAUNCH_ST = rv_launch(kernel, dim3(n_tokens), dim3(QP_WARPS * 32), 0, stream, a);
+    return rv_launch_status();
+}
+
+// ------------------------------------------------------------------ after the attention kernels
+// V neighbouring elements per thread and access: 4 (8 or 16 bytes) where sizes and pointers allow, else 1.
+template <int V>
+__device__ __forceinline__ void qp_load_vec(const void* p, int dtype, size_t i, float (&v)[V]) {
+    if constexpr (V == 4) {
+        if (dtype == RV_DTYPE_F32) {
+            const float4 f = *reinterpret_cast<const float4*>((const float*)p + i);
+            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+        } else {
+            const uint2 u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
+            const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+            const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+            v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+        }
+    } else {
+        v[0] = dtype == RV_DTYPE_F32 ? ((const float*)p)[i] : __bfloat162float(((const __nv_bfloat16*)p)[i]);
+    }
+}
+template <int V>
+__device__ __forceinline__ void qp_store_vec(void* p, int dtype, size_t i, const float (&v)[V]) {
+    if constexpr (V == 4) {
+        if (dtype == RV_DTYPE_F32) {
+            *reinterpret_cast<float4*>((float*)p + i) = make_float4(v[0], v[1], v[2], v[3]);
+        } else {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+            uint2 u;
+            u.x = *reinterpret_cast<uint32_t*>(&lo); u.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>((__nv_bfloat16*)p + i) = u;
+        }
+    } else {
+        qp_store(p, dtype, i, v[0]);
+    }
+}
+
+// A thread takes V neighbouring pairs.  halves: pairs (m, m + vd / 2); else (2m, 2m + 1), V = 1.
+template <int V>
+__global__ void __launch_bounds__(256)
+turn_back_kernel(const void* __restrict__ o, const int* __restrict__ positions, const float* __restrict__ cos_t,
+                 const float* __restrict__ sin_t, int table_rows, int halves, void* __restrict__ out, int dtype, int nh, int vd, int P,
+                 size_t total) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    const int half = vd >> 1, per_head = half / V, per_token = per_head * nh;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = i / per_token;
+        const int in_token = (int)(i - t * per_token), h = in_token / per_head, m = (in_token - h * per_head) * V;
+        int pos = positions[t];
+        if (pos < 0) pos = 0;
+        if (pos >= table_rows) pos = table_rows - 1;
+        const size_t src = (t * nh + h) * P, dst = (t * nh + h) * vd;
+        const int first = halves ? m : 2 * m, second = halves ? m + half : 2 * m + 1;
+        float a[V], b[V], c[V], s[V], u[V], w[V];
+        qp_load_vec<V>(o, dtype, src + first, a);
+        qp_load_vec<V>(o, dtype, src + second, b);
+        qp_load_vec<V>(cos_t, RV_DTYPE_F32, (size_t)pos * half + m, c);
+        qp_load_vec<V>(sin_t, RV_DTYPE_F32, (size_t)pos * half + m, s);
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+            u[j] = a[j] * c[j] + b[j] * s[j];
+            w[j] = b[j] * c[j] - a[j] * s[j];
+        }
+        qp_store_vec<V>(out, dtype, dst + first, u);
+        qp_store_vec<V>(out, dtype, dst + second, w);
+    }
+}
+
+static inline int qp_blocks(size_t items) {
+    const size_t want = (items + 255) / 256;
+    return (int)(want < 148 * 16 ? (want ? want : 1) : 148 * 16);
+}
+
+RV_EXPORT int rv_turn_back(const void* o, const int* positions, const float* cos_t, const float* sin_t, int table_rows, int halves,
+                           void* out, int dtype, int n_tokens, int nh, int vd, int P, cudaStream_t stream) {
+    if (n_tokens < 0 || nh <= 0 || vd <= 0 || (vd & 1) || P < vd || table_rows <= 0) return RV_ERR_BAD_SIZE;
+    if (dtype & ~1) return RV_ERR_BAD_DTYPE;
+    if (n_tokens == 0) return RV_OK;
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(cos_t) |
+                           reinterpret_cast<uintptr_t>(sin_t);
+    const size_t pairs = (size_t)n_tokens * nh * (vd / 2);
+    if (halves && vd % 8 == 0 && P % 4 == 0 && bits % 16 == 0)
+        RV_LAUNCH_ST = rv_launch(turn_back_kernel<4>, dim3(qp_blocks(pairs / 4)), dim3(256), 0, stream, o, positions, cos_t, sin_t,
+                                 table_rows, halves, out, dtype, nh, vd, P, pairs / 4);
+    else
+        RV_LAUNCH_ST = rv_launch(turn_back_kernel<1>, dim3(qp_blocks(pairs)), dim3(256), 0, stream, o, positions, cos_t, sin_t,
+                                 table_rows, halves, out, dtype, nh, vd, P, pairs);
+    return rv_launch_status();
+}
+
+// One warp per (token, head); a head's vd elements in NJ accesses of V per lane (vd <= 32 V NJ).
+template <int V, int NJ>
+__global__ void __launch_bounds__(256)
+map_difference_kernel(const void* __restrict__ o, float lambda, float eps, float factor, void* __restrict__ out, int dtype, int vd,
+                      int P, size_t total_heads) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const size_t w = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (w >= total_heads) return;
+    const size_t first = w * 2 * P, second = first + P;
+    float v[NJ][V];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        const int i = (j * 32 + lane) * V;
+        if (i < vd) {
+            float b[V];
+            qp_load_vec<V>(o, dtype, first + i, v[j]);
+            qp_load_vec<V>(o, dtype, second + i, b);
+#pragma unroll
+            for (int k = 0; k < V; ++k) {
+                v[j][k] = fmaf(-lambda, b[k], v[j][k]);
+                ss = fmaf(v[j][k], v[j][k], ss);
+            }
+        }
+    }
+    ss = rv_warp_sum(ss);
+    const float r = factor / sqrtf(ss / (float)vd + eps);
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        const int i = (j * 32 + lane) * V;
+        if (i < vd) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) v[j][k] *= r;
+            qp_store_vec<V>(out, dtype, w * vd + i, v[j]);
+        }
+    }
+}
+
+RV_EXPORT int rv_map_difference(const void* o, float lambda, float eps, float factor, void* out, int dtype, int n_tokens, int nh, int vd,
+                                int P, cudaStream_t stream) {
+    if (n_tokens < 0 || nh <= 0 || vd <= 0 || P < vd) return RV_ERR_BAD_SIZE;
+    if (vd > QP_MAX_DIM) return RV_ERR_UNSUPPORTED;
+    if (dtype & ~1) return RV_ERR_BAD_DTYPE;
+    if (n_tokens == 0) return RV_OK;
+    const size_t total = (size_t)n_tokens * nh;
+    const dim3 grid((unsigned)((total + 7) / 8));
+    const bool vec = vd % 4 == 0 && P % 4 == 0 && ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(out)) % 16) == 0;
+    auto kernel = vec ? (vd <= 128 ? map_difference_kernel<4, 1> : (vd <= 256 ? map_difference_kernel<4, 2> : map_difference_kernel<4, 8>))
+                      : (vd <= 128 ? map_difference_kernel<1, 4> : (vd <= 256 ? map_difference_kernel<1, 8> : map_difference_kernel<1, 32>));
+    RV_LAUNCH_ST = rv_launch(kernel, grid, dim3(256), 0, stream, o, lambda, eps, factor, out, dtype, vd, P, total);
     return rv_launch_status();
 }

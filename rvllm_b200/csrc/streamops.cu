@@ -15,6 +15,10 @@
 //                         new x with a second (alpha, w, b), in the activations' type: the next sublayer's input
 //   scale_rows            x * s as float32 (the start of a float32 stream from a table kept in 16 bits)
 //   act_rows              relu(u)^2, optionally times one number per row, in the activations' type
+//   stream_combine        x += sum of up to three float32 terms, each with a factor, and up to two RMSNorms of the new x
+//                         from one row statistic (the inputs of sublayers that stand side by side)
+//   bigram_add            x + table[hash of (previous token, token)] as float32 (the start of a float32 stream); the last
+//                         token of a sequence's share is kept in its state row for the next step
 //
 // All arithmetic is float (the angle: double); storage is float or bfloat16 per argument.  Any width.
 #include "common.cuh"
@@ -370,5 +374,176 @@ RV_EXPORT int rv_act_rows(const void* u, int u_dtype, const float* row_scale, vo
                                  cols, total / 4);
     else
         RV_LAUNCH_ST = rv_launch(act_rows_kernel, dim3(so_blocks(total)), dim3(256), 0, stream, u, u_dtype, row_scale, out, out_dtype, cols, total);
+    return rv_launch_status();
+}
+
+// ------------------------------------------------------------------ stream += weighted terms, and the norms of the new stream
+struct CombineArgs {
+    float* x;
+    const float* y[3]; float c[3]; int terms;
+    const void* gamma[2]; int gamma_dtype[2]; float eps[2]; int norms;
+    void* out[2]; int out_dtype;
+    int cols;
+};
+
+// A row per block.  NV > 0: 4 columns a thread and access, the row in NV accesses per thread held in registers
+// (cols = 4 * blockDim * NV at most); NV = 0: any width, the row is read again for the norms.
+template <int NV>
+__global__ void __launch_bounds__(256)
+stream_combine_kernel(const CombineArgs a) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    __shared__ float scratch[33];
+    const size_t base = (size_t)blockIdx.x * a.cols;
+    float ss = 0.f;
+    if constexpr (NV > 0) {
+        float4 v[NV];
+        const int quads = a.cols / 4;
+        float4* x4 = reinterpret_cast<float4*>(a.x + base);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            if (i < quads) v[j] = x4[i];
+        }
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            if (k >= a.terms) break;
+            const float4* y4 = reinterpret_cast<const float4*>(a.y[k] + base);
+            const float c = a.c[k];
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int i = threadIdx.x + j * blockDim.x;
+                if (i < quads) {
+                    const float4 y = y4[i];
+                    v[j].x = fmaf(c, y.x, v[j].x); v[j].y = fmaf(c, y.y, v[j].y);
+                    v[j].z = fmaf(c, y.z, v[j].z); v[j].w = fmaf(c, y.w, v[j].w);
+                }
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            if (i < quads) {
+                if (a.terms) x4[i] = v[j];
+                ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+            }
+        }
+        if (a.norms == 0) return;
+        ss = rv_block_sum(ss, scratch);
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            if (k >= a.norms) break;
+            const float r = 1.0f / sqrtf(ss / (float)a.cols + a.eps[k]);
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int i = threadIdx.x + j * blockDim.x;
+                if (i >= quads) continue;
+                float4 g;
+                if (a.gamma_dtype[k] == RV_DTYPE_F32) {
+                    g = reinterpret_cast<const float4*>(a.gamma[k])[i];
+                } else {
+                    const uint2 u = reinterpret_cast<const uint2*>(a.gamma[k])[i];
+                    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+                    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+                    g = make_float4(lo.x, lo.y, hi.x, hi.y);
+                }
+                const float o0 = v[j].x * r * g.x, o1 = v[j].y * r * g.y, o2 = v[j].z * r * g.z, o3 = v[j].w * r * g.w;
+                if (a.out_dtype == RV_DTYPE_F32) {
+                    reinterpret_cast<float4*>((float*)a.out[k] + base)[i] = make_float4(o0, o1, o2, o3);
+                } else {
+                    __nv_bfloat162 lo = __floats2bfloat162_rn(o0, o1), hi = __floats2bfloat162_rn(o2, o3);
+                    uint2 pk;
+                    pk.x = *reinterpret_cast<uint32_t*>(&lo); pk.y = *reinterpret_cast<uint32_t*>(&hi);
+                    reinterpret_cast<uint2*>((__nv_bfloat16*)a.out[k] + base)[i] = pk;
+                }
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < a.cols; i += blockDim.x) {
+            float v = a.x[base + i];
+#pragma unroll
+            for (int k = 0; k < 3; ++k)
+                if (k < a.terms) v = fmaf(a.c[k], a.y[k][base + i], v);
+            if (a.terms) a.x[base + i] = v;
+            ss = fmaf(v, v, ss);
+        }
+        if (a.norms == 0) return;
+        ss = rv_block_sum(ss, scratch);
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            if (k >= a.norms) break;
+            const float r = 1.0f / sqrtf(ss / (float)a.cols + a.eps[k]);
+            for (int i = threadIdx.x; i < a.cols; i += blockDim.x)        // every thread reads back what it wrote itself
+                so_store(a.out[k], a.out_dtype, base + i, a.x[base + i] * r * rv_load_param(a.gamma[k], a.gamma_dtype[k], i));
+        }
+    }
+}
+
+// terms: y0 .. y2 with factors c0 .. c2, the first null one ends them; norms: gamma0, gamma1 likewise (out0, out1 their results).
+RV_EXPORT int rv_stream_combine(float* x, const float* y0, float c0, const float* y1, float c1, const float* y2, float c2,
+                                const void* gamma0, int g0_dtype, float eps0, void* out0, const void* gamma1, int g1_dtype, float eps1,
+                                void* out1, int out_dtype, int rows, int cols, cudaStream_t stream) {
+    if (rows < 0 || cols <= 0) return RV_ERR_BAD_SIZE;
+    if ((g0_dtype | g1_dtype | out_dtype) & ~1) return RV_ERR_BAD_DTYPE;
+    CombineArgs a = {x, {y0, y1, y2}, {c0, c1, c2}, y0 ? (y1 ? (y2 ? 3 : 2) : 1) : 0, {gamma0, gamma1}, {g0_dtype, g1_dtype},
+                     {eps0, eps1}, gamma0 ? (gamma1 ? 2 : 1) : 0, {out0, out1}, out_dtype, cols};
+    if ((a.norms > 0 && !out0) || (a.norms > 1 && !out1)) return RV_ERR_BAD_SIZE;
+    if (rows == 0 || (a.terms == 0 && a.norms == 0)) return RV_OK;
+    uintptr_t bits = reinterpret_cast<uintptr_t>(x);
+    for (int k = 0; k < a.terms; ++k) bits |= reinterpret_cast<uintptr_t>(a.y[k]);
+    for (int k = 0; k < a.norms; ++k) bits |= reinterpret_cast<uintptr_t>(a.gamma[k]) | reinterpret_cast<uintptr_t>(a.out[k]);
+    const int threads = cols >= 1024 ? 256 : 128;
+    const int nv = (cols / 4 + threads - 1) / threads;
+    auto kernel = stream_combine_kernel<0>;
+    if (cols % 4 == 0 && bits % 16 == 0 && nv <= 8)
+        kernel = nv <= 1 ? stream_combine_kernel<1> : (nv <= 2 ? stream_combine_kernel<2> : (nv <= 4 ? stream_combine_kernel<4>
+                                                                                                  : stream_combine_kernel<8>));
+    RV_LAUNCH_ST = rv_launch(kernel, dim3(rows), dim3(threads), 0, stream, a);
+    return rv_launch_status();
+}
+
+// ------------------------------------------------------------------ bigram rows
+// A block per token.  The row is (previous token * mul_prev + token * mul_cur) mod buckets, and `buckets` for position 0.  The
+// previous token of a share's first token comes from the sequence's state row; the block of that token - the only one
+// that reads the state - also leaves the share's last token there.
+__global__ void __launch_bounds__(256)
+bigram_add_kernel(const void* __restrict__ x, int x_dtype, const void* __restrict__ table, int table_dtype, const int* __restrict__ ids,
+                  const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens,
+                  const int* __restrict__ state_slots, int* __restrict__ state, int state_stride, long long mul_prev, long long mul_cur,
+                  int buckets, float* __restrict__ out, int cols) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    __shared__ int row_s;
+    const int t = blockIdx.x;
+    if (threadIdx.x == 0) {
+        const int seq = token_seq[t];
+        const int first = seq >= 0 ? cu_seqlens[seq] : t;
+        const int slot = seq >= 0 ? state_slots[seq] : -1;
+        int prev = 0;
+        if (t > first) prev = ids[t - 1];
+        else if (slot >= 0) prev = state[(size_t)slot * state_stride];
+        long long r = buckets;
+        if (positions[t] > 0) {
+            r = ((long long)prev * mul_prev + (long long)ids[t] * mul_cur) % buckets;
+            if (r < 0) r += buckets;
+        }
+        row_s = (int)r;
+        if (t == first && slot >= 0) state[(size_t)slot * state_stride] = ids[cu_seqlens[seq + 1] - 1];
+    }
+    __syncthreads();
+    const size_t src = (size_t)row_s * cols, dst = (size_t)t * cols;
+    for (int i = threadIdx.x; i < cols; i += blockDim.x) out[dst + i] = so_load(x, x_dtype, dst + i) + so_load(table, table_dtype, src + i);
+}
+
+// state int rows of `state_stride`; table [buckets + 1, cols]; mul_prev and mul_cur are taken modulo `buckets` by the caller.
+RV_EXPORT int rv_bigram_add(const void* x, int x_dtype, const void* table, int table_dtype, const int* ids, const int* positions,
+                            const int* token_seq, const int* cu_seqlens, const int* state_slots, int* state, int state_stride,
+                            long long mul_prev, long long mul_cur, int buckets, float* out, int rows, int cols, cudaStream_t stream) {
+    if (rows < 0 || cols <= 0 || buckets <= 0 || state_stride <= 0) return RV_ERR_BAD_SIZE;
+    if ((x_dtype | table_dtype) & ~1) return RV_ERR_BAD_DTYPE;
+    if (mul_prev < 0 || mul_prev >= buckets || mul_cur < 0 || mul_cur >= buckets) return RV_ERR_BAD_SIZE;      // the sum stays below 2^63
+    if (rows == 0) return RV_OK;
+    RV_LAUNCH_ST = rv_launch(bigram_add_kernel, dim3(rows), dim3(cols >= 1024 ? 256 : 128), 0, stream, x, x_dtype, table, table_dtype, ids,
+                             positions, token_seq, cu_seqlens, state_slots, state, state_stride, mul_prev, mul_cur, buckets, out, cols);
     return rv_launch_status();
 }

@@ -38,10 +38,11 @@ class StepEntry:
 class StepContext:
     """What the parts see of a step."""
     __slots__ = ("kernels", "num_tokens", "num_seqs", "token_ids", "positions", "token_seq", "cu_seqlens",
-                 "state_slots", "logit_rows", "attention", "q_lens", "ctx_lens", "req_ids", "extras")
+                 "state_slots", "logit_rows", "attention", "q_lens", "ctx_lens", "req_ids", "extras", "following_norms")
 
     def __init__(self):
         self.extras = {}
+        self.following_norms = None      # the norms in front of the block that runs next, if this block may form them (parts/base.py)
 
 
 class ModelRunner:

@@ -482,11 +482,11 @@ class CudaKernels:
         _need(q, "q", dims=2); _need(cache_layer, "cache_layer", q.dtype, 5)
         self._check_attention_extras(q, num_heads, sinks, gate)
         out = torch.empty_like(q)
-        st = self._lib("attention_ref.cu").rv_paged_attention_ref(
+        st = self._lib("attention_ref.cu").rv_paged_attention_ref_ex(
             _ptr(q), _ptr(cache_layer), _ptr(meta.block_tables), _ptr(meta.cu_seqlens), _ptr(meta.ctx_lens),
             _ptr(meta.token_seq), _ptr(out), c_int(q.shape[0]), c_int(num_heads), c_int(num_kv_heads),
-            c_int(head_dim), c_int(cache_layer.shape[3]), c_int(meta.max_blocks), c_float(scale),
-            c_int(window or 0), c_float(softcap or 0.0), _ptr(sinks), _ptr(gate), c_int(self._dt(q, "q")), self._stream())
+            c_int(head_dim), c_int(cache_layer.shape[3]), c_int(meta.max_blocks), c_float(scale), c_int(window or 0),
+            c_float(softcap or 0.0), _ptr(sinks), _ptr(gate), c_int(2), c_int(head_dim), c_int(self._dt(q, "q")), self._stream())
         _check("paged_attention_plain", st)
         return out
 
@@ -1452,11 +1452,13 @@ class CudaKernels:
 
     # ------------------------------------------------------------------ mixture of experts
     def moe_experts(self, x, chosen, gate_up, down, weight: float, add: Optional[torch.Tensor] = None, out_dtype=None,
-                    weights: Optional[torch.Tensor] = None, activation: str = "silu") -> torch.Tensor:
-        """out[t] = (add[t]) + weight * sum_k weights[t, k] down[e] a_e(x_t), e = chosen[t, k].
+                    weights: Optional[torch.Tensor] = None, activation: str = "silu",
+                    add_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """out[t] = (add_scale[t] * add[t]) + weight * sum_k weights[t, k] down[e] a_e(x_t), e = chosen[t, k].
         activation "silu": gated experts, a_e(x) = silu(gate[e] x) * (up[e] x), gate_up [experts, 2 ff, width] (gate rows, then up
         rows); "relu2": plain experts, a_e(x) = relu(up[e] x)^2, `gate_up` is up [experts, ff, width].  down [experts, width, ff],
-        chosen int32 [T, top], weights float32 [T, top] or None (all 1), add float32 [T, width] or None."""
+        chosen int32 [T, top], weights float32 [T, top] or None (all 1), add float32 [T, width] or None,
+        add_scale float32 [T] or None (all 1)."""
         _need(x, "x", dims=2); _need(chosen, "chosen", torch.int32, 2)
         _need(gate_up, "gate_up", x.dtype, 3); _need(down, "down", x.dtype, 3)
         if activation not in ("silu", "relu2"):
@@ -1476,16 +1478,20 @@ class CudaKernels:
             _need(add, "add", torch.float32, 2)
             if add.shape != x.shape:
                 raise KernelError(f"moe_experts: add {tuple(add.shape)} against x {tuple(x.shape)}")
+        if add_scale is not None:
+            _need(add_scale, "add_scale", torch.float32, 1)
+            if add is None or add_scale.shape[0] != T:
+                raise KernelError(f"moe_experts: {add_scale.shape[0]} factors on what is added to {T} rows")
         out_dtype = out_dtype or x.dtype
         if out_dtype not in (x.dtype, torch.float32):
             raise KernelError(f"moe_experts: result type {out_dtype} for operands of {x.dtype}")
         if x.dtype == torch.bfloat16 and T >= self.MOE_GROUPED_MIN_TOKENS and width % 8 == 0 and ff % 8 == 0 and E <= 4096:
-            return self._moe_grouped(x, chosen, gate_up, down, weight, add, out_dtype, weights, gated)
+            return self._moe_grouped(x, chosen, gate_up, down, weight, add, out_dtype, weights, gated, add_scale)
         act = torch.empty((T * top, ff), dtype=x.dtype, device=x.device)
         out = torch.empty((T, width), dtype=out_dtype, device=x.device)
         st = self._lib("moe.cu").rv_moe_experts_ex(
-            _ptr(x), _ptr(chosen), _ptr(weights), _ptr(gate_up), _ptr(down), _ptr(act), _ptr(add), _ptr(out),
-            c_int(1 if out_dtype == torch.float32 else 0), c_int(T), c_int(top), c_int(E), c_int(ff), c_int(width), c_float(weight),
+            _ptr(x), _ptr(chosen), _ptr(weights), _ptr(gate_up), _ptr(down), _ptr(act), _ptr(add), _ptr(add_scale),
+            _ptr(out), c_int(1 if out_dtype == torch.float32 else 0), c_int(T), c_int(top), c_int(E), c_int(ff), c_int(width), c_float(weight),
             c_int(1 if gated else 0), c_int(self._dt(x, "x")), self._stream())
         _check("moe_experts", st)
         COUNTERS['launches'] += 1
@@ -1494,7 +1500,7 @@ class CudaKernels:
     MOE_GROUPED_MIN_TOKENS = 128      # tokens of a step from which the experts' products run grouped on the tcgen05 GEMM ...
     MOE_GROUPED_PAIRS = True          # ... on pairs of CTAs (cta_group::2): two blocks of 128 rows of one expert share every tile of its weights
 
-    def _moe_grouped(self, x, chosen, gate_up, down, weight, add, out_dtype, weights=None, gated=True):
+    def _moe_grouped(self, x, chosen, gate_up, down, weight, add, out_dtype, weights=None, gated=True, add_scale=None):
         """`moe_experts` for many bfloat16 tokens: the (token, slot) pairs sorted by expert, every expert's rows padded to
         whole blocks of 128, two grouped tcgen05 products over the sorted rows (gate/up with the SiLU epilogue - plain experts:
         up with the squared relu in its epilogue - then down with a float32 result), and the weighted sum per token.  Everything is decided on the device; the buffers are sized for the worst case (every
@@ -1533,15 +1539,19 @@ class CudaKernels:
             c_int(units), c_int(0), _ptr(self._status), self._stream()))
         out = torch.empty((T, width), dtype=out_dtype, device=dev)
         _check("moe_combine", moe.rv_moe_combine(_ptr(ys), _ptr(row_of), _ptr(add), _ptr(out), c_int(1 if out_dtype == torch.float32 else 0),
-                                                 c_int(T), c_int(top), c_int(width), c_float(weight), _ptr(weights), self._stream()))
+                                                 c_int(T), c_int(top), c_int(width), c_float(weight), _ptr(weights), _ptr(add_scale),
+                                                 self._stream()))
         return out
 
     def moe_route_top(self, scores, correction, experts: int, top: int, groups: int, keep: int, weight_eps: float,
-                      shared_gate: bool = False):
+                      shared_gate: bool = False, scoring: str = "sigmoid"):
         """A router's choice from its float32 logits [T, experts (+ 1)]: s = sigmoid(logits); the `top` experts with the largest
         s + correction among those of the `keep` best of `groups` equal groups of neighbouring experts (a group counts by the
         sum of its two largest corrected scores).  Returns (chosen int32 [T, top], weights float32 [T, top] = the chosen s over
-        their sum + weight_eps, sigmoid of the last column float32 [T] with `shared_gate`, else None)."""
+        their sum + weight_eps, sigmoid of the last column float32 [T] with `shared_gate`, else None).  scoring "softmax": the choice
+        is made among logits + correction, and the weights are the softmax over the chosen ones (then divided by 1 + weight_eps / sum)."""
+        if scoring not in ("sigmoid", "softmax"):
+            raise KernelError(f"moe_route_top: scoring {scoring!r} is not known (sigmoid, softmax)")
         _need(scores, "scores", torch.float32, 2); _need(correction, "correction", torch.float32, 1)
         T = scores.shape[0]
         if scores.shape[1] != experts + (1 if shared_gate else 0) or correction.shape[0] != experts:
@@ -1551,7 +1561,7 @@ class CudaKernels:
         gate = torch.empty((T,), dtype=torch.float32, device=scores.device) if shared_gate else None
         st = self._lib("moe.cu").rv_moe_route_top(
             _ptr(scores), c_int(scores.shape[1]), _ptr(correction), _ptr(chosen), _ptr(weights), _ptr(gate), c_int(T), c_int(experts),
-            c_int(top), c_int(groups), c_int(keep), c_float(weight_eps), self._stream())
+            c_int(top), c_int(groups), c_int(keep), c_float(weight_eps), c_int(1 if scoring == "softmax" else 0), self._stream())
         _check("moe_route_top", st)
         return chosen, weights, gate
 
@@ -1615,42 +1625,162 @@ class CudaKernels:
         return out
 
     # ------------------------------------------------------------------ unit-norm attention, mLSTM
-    def qk_unit_prepare(self, proj, eps: float, positions, cos, sin, slot_mapping, cache_layer, num_heads: int, num_kv_heads: int,
-                        head_dim: int, value_dim: int, slot_dim: int, out_dtype, halves: bool = False, with_gate: bool = True,
-                        write_kv: bool = True):
-        """proj float32 rows [q: heads x head_dim | k: kv heads x head_dim | v: kv heads x value_dim | gate logits: heads] (k and v
-        only with `write_kv`).  q and k: the leading 2 * cos.shape[1] elements of every head turn in pairs (2i, 2i + 1) - with
-        `halves`: (i, i + cos.shape[1]) -, then the head is divided by sqrt(mean(x^2) + eps).  k and v go into the token's
-        cache slot, in heads of `slot_dim` elements whose tail is zeros.  Returns (q [T, heads * slot_dim] in `out_dtype`,
-        sigmoid(gate logits) float32 [T, heads] or None)."""
+    def qk_prepare(self, proj, positions, cos, sin, slot_mapping, cache_layer, num_heads: int, num_kv_heads: int, head_dim: int,
+                   value_dim: int, slot_dim: int, out_dtype, eps: Optional[float] = None, halves: bool = False, with_gate: bool = False,
+                   write_kv: bool = True, maps: int = 1, bias: Optional[torch.Tensor] = None, value_tables=None):
+        """proj float32 rows [q: heads x maps x head_dim | k: kv heads x maps x head_dim | v: kv heads x value_dim | gate logits:
+        heads] (k and v only with `write_kv`), plus `bias` (float32, a number per column of q, k and v).  q and k: the leading
+        2 * cos.shape[1] elements of every map turn in pairs (2i, 2i + 1) - with `halves`: (i, i + cos.shape[1]) -, then, with
+        `eps`, the map is divided by sqrt(mean(x^2) + eps).  value_tables = (cos, sin) [rows, value_dim / 2]: v turns too, over
+        all its elements.  k (its maps side by side) and v go into the token's cache slot, in heads of `slot_dim` elements
+        whose tail is zeros; a query row of map m holds its elements at m * head_dim and zeros elsewhere, so that its product
+        with the key row is map m's score.  Returns (q [T, heads * maps * slot_dim] in `out_dtype`, sigmoid(gate logits)
+        float32 [T, heads] or None)."""
         _need(proj, "proj", torch.float32, 2); _need(positions, "positions", torch.int32, 1)
         T = proj.shape[0]
-        want = num_heads * head_dim + (num_kv_heads * (head_dim + value_dim) if write_kv else 0) + (num_heads if with_gate else 0)
-        if proj.shape[1] != want or slot_dim < max(head_dim, value_dim):
-            raise KernelError(f"qk_unit_prepare: rows of {proj.shape[1]} columns do not fit {num_heads} heads of {head_dim}"
-                              + (f", {num_kv_heads} key/value heads of {head_dim} / {value_dim}" if write_kv else "")
+        cols = maps * num_heads * head_dim + (num_kv_heads * (maps * head_dim + value_dim) if write_kv else 0)
+        if proj.shape[1] != cols + (num_heads if with_gate else 0) or slot_dim < max(maps * head_dim, value_dim):
+            raise KernelError(f"qk_prepare: rows of {proj.shape[1]} columns do not fit {num_heads} heads of {maps} x {head_dim}"
+                              + (f", {num_kv_heads} key/value heads of {maps} x {head_dim} / {value_dim}" if write_kv else "")
                               + (f" and {num_heads} gates" if with_gate else "") + f" in slots of {slot_dim}")
         rot, table_rows = 0, 1
         if cos is not None:
             _need(cos, "cos", torch.float32, 2); _need(sin, "sin", torch.float32, 2)
             rot, table_rows = 2 * cos.shape[1], cos.shape[0]
             if not 0 < rot <= head_dim or sin.shape != cos.shape:
-                raise KernelError(f"qk_unit_prepare: cos/sin tables must be [rows, dims/2] with dims <= {head_dim}")
+                raise KernelError(f"qk_prepare: cos/sin tables must be [rows, dims/2] with dims <= {head_dim}")
+        vcos, vsin = value_tables if value_tables is not None else (None, None)
+        if vcos is not None:
+            _need(vcos, "value cos", torch.float32, 2); _need(vsin, "value sin", torch.float32, 2)
+            if 2 * vcos.shape[1] != value_dim or vsin.shape != vcos.shape:
+                raise KernelError(f"qk_prepare: value tables {tuple(vcos.shape)} for values of {value_dim}")
+        if bias is not None:
+            _need(bias, "bias", torch.float32, 1)
+            if bias.shape[0] != cols:
+                raise KernelError(f"qk_prepare: {bias.shape[0]} biases for {cols} columns")
         page = 1
         if write_kv:
             _need(cache_layer, "cache_layer", out_dtype, 5); _need(slot_mapping, "slot_mapping", torch.int32, 1)
             if cache_layer.shape[1] != 2 or cache_layer.shape[2] != num_kv_heads or cache_layer.shape[4] != slot_dim:
-                raise KernelError(f"qk_unit_prepare: cache layer of shape {tuple(cache_layer.shape)} for {num_kv_heads} heads of {slot_dim}")
+                raise KernelError(f"qk_prepare: cache layer of shape {tuple(cache_layer.shape)} for {num_kv_heads} heads of {slot_dim}")
             page = cache_layer.shape[3]
-        q = torch.empty((T, num_heads * slot_dim), dtype=out_dtype, device=proj.device)
+        q = torch.empty((T, num_heads * maps * slot_dim), dtype=out_dtype, device=proj.device)
         gate = torch.empty((T, num_heads), dtype=torch.float32, device=proj.device) if with_gate else None
-        st = self._lib("qk_prepare.cu").rv_qk_unit_prepare(
-            _ptr(proj), c_int(proj.shape[1]), _ptr(positions), _ptr(cos), _ptr(sin), c_int(rot), c_int(table_rows),
-            c_int(1 if halves else 0), _ptr(slot_mapping if write_kv else None), _ptr(cache_layer if write_kv else None), _ptr(q),
-            c_int(_DT[out_dtype]), _ptr(gate), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(value_dim),
-            c_int(slot_dim), c_int(page), c_float(eps), c_int(1 if write_kv else 0), self._stream())
-        _check("qk_unit_prepare", st)
+        st = self._lib("qk_prepare.cu").rv_qk_prepare(
+            _ptr(proj), c_int(proj.shape[1]), _ptr(bias), _ptr(positions), _ptr(cos), _ptr(sin), c_int(rot), c_int(table_rows),
+            c_int(1 if halves else 0), _ptr(vcos), _ptr(vsin), c_int(vcos.shape[0] if vcos is not None else 1),
+            _ptr(slot_mapping if write_kv else None), _ptr(cache_layer if write_kv else None), _ptr(q), c_int(_DT[out_dtype]), _ptr(gate),
+            c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(value_dim), c_int(slot_dim), c_int(maps), c_int(page),
+            c_float(eps or 0.0), c_int(1 if eps is not None else 0), c_int(1 if write_kv else 0), self._stream())
+        _check("qk_prepare", st)
         return q, gate
+
+    def qk_unit_prepare(self, proj, eps: float, positions, cos, sin, slot_mapping, cache_layer, num_heads: int, num_kv_heads: int,
+                        head_dim: int, value_dim: int, slot_dim: int, out_dtype, halves: bool = False, with_gate: bool = True,
+                        write_kv: bool = True, value_tables=None):
+        """`qk_prepare` for one map per head, with the unit norm on q and k."""
+        return self.qk_prepare(proj, positions, cos, sin, slot_mapping, cache_layer, num_heads, num_kv_heads, head_dim, value_dim,
+                               slot_dim, out_dtype, eps=eps, halves=halves, with_gate=with_gate, write_kv=write_kv,
+                               value_tables=value_tables)
+
+    def turn_back(self, o, positions, cos, sin, heads: int, value_dim: int, slot_dim: int, halves: bool = True) -> torch.Tensor:
+        """The leading `value_dim` elements of every head of o [T, heads * slot_dim], turned by minus the token's angle in pairs
+        (m, m + value_dim / 2) - without `halves`: (2m, 2m + 1); tables [rows, value_dim / 2].  Returns [T, heads * value_dim]."""
+        _need(o, "o", dims=2); _need(positions, "positions", torch.int32, 1)
+        _need(cos, "cos", torch.float32, 2); _need(sin, "sin", torch.float32, 2)
+        T = o.shape[0]
+        if o.shape[1] != heads * slot_dim or slot_dim < value_dim or 2 * cos.shape[1] != value_dim or sin.shape != cos.shape:
+            raise KernelError(f"turn_back: rows of {o.shape[1]}, tables {tuple(cos.shape)} for {heads} heads of {value_dim} in slots of {slot_dim}")
+        out = torch.empty((T, heads * value_dim), dtype=o.dtype, device=o.device)
+        st = self._lib("qk_prepare.cu").rv_turn_back(
+            _ptr(o), _ptr(positions), _ptr(cos), _ptr(sin), c_int(cos.shape[0]), c_int(1 if halves else 0), _ptr(out), c_int(self._dt(o, "o")),
+            c_int(T), c_int(heads), c_int(value_dim), c_int(slot_dim), self._stream())
+        _check("turn_back", st)
+        return out
+
+    def map_difference(self, o, lam: float, eps: float, factor: float, heads: int, value_dim: int, slot_dim: int) -> torch.Tensor:
+        """o [T, heads * 2 * slot_dim] holds two maps' results per head: d = a1 - lam * a2 over their leading `value_dim` elements,
+        then factor * d / sqrt(mean(d^2) + eps).  Returns [T, heads * value_dim]."""
+        _need(o, "o", dims=2)
+        T = o.shape[0]
+        if o.shape[1] != heads * 2 * slot_dim or slot_dim < value_dim:
+            raise KernelError(f"map_difference: rows of {o.shape[1]} for {heads} heads of 2 x {value_dim} in slots of {slot_dim}")
+        out = torch.empty((T, heads * value_dim), dtype=o.dtype, device=o.device)
+        st = self._lib("qk_prepare.cu").rv_map_difference(_ptr(o), c_float(lam), c_float(eps), c_float(factor), _ptr(out),
+                                                          c_int(self._dt(o, "o")), c_int(T), c_int(heads), c_int(value_dim),
+                                                          c_int(slot_dim), self._stream())
+        _check("map_difference", st)
+        return out
+
+    # ------------------------------------------------------------------ sublayers side by side, minGRU, bigram rows
+    def stream_combine(self, x, terms, norms, out_dtype):
+        """x += sum of c * y over terms [(y, c), ...] (up to three, float32) on the float32 stream, in place; then, for each
+        (gamma, eps) of `norms` (up to two), the new x / sqrt(mean(x^2) + eps) * gamma in `out_dtype`, all from one row
+        statistic.  Returns (x, [normalised rows, ...])."""
+        _need(x, "x", torch.float32, 2)
+        rows, cols = x.shape
+        if len(terms) > 3 or len(norms) > 2:
+            raise KernelError(f"stream_combine: {len(terms)} terms and {len(norms)} norms (at most three and two)")
+        for y, _ in terms:
+            _need(y, "y", torch.float32, 2)
+            if y.shape != x.shape:
+                raise KernelError(f"stream_combine: {tuple(y.shape)} added to {tuple(x.shape)}")
+        for gamma, _ in norms:
+            _need(gamma, "gamma", dims=1)
+            if gamma.shape[0] != cols:
+                raise KernelError(f"stream_combine: gamma has {gamma.shape[0]} entries for rows of {cols}")
+        if not terms and not norms:
+            return x, []
+        outs = [torch.empty((rows, cols), dtype=out_dtype, device=x.device) for _ in norms]
+        args = []
+        for i in range(3):
+            y, c = terms[i] if i < len(terms) else (None, 0.0)
+            args += [_ptr(y), c_float(c)]
+        for i in range(2):
+            gamma, eps = norms[i] if i < len(norms) else (None, 0.0)
+            args += [_ptr(gamma), c_int(self._dt(gamma, "gamma") if gamma is not None else 0), c_float(eps), _ptr(outs[i] if i < len(outs) else None)]
+        st = self._lib("streamops.cu").rv_stream_combine(_ptr(x), *args, c_int(_DT[out_dtype] if outs else 0), c_int(rows), c_int(cols),
+                                                         self._stream())
+        _check("stream_combine", st)
+        return x, outs
+
+    def mingru(self, proj, z_bias, x_bias, cu_seqlens, state_slots, state, width: int, single: bool, out_dtype) -> torch.Tensor:
+        """The minGRU recurrence over the step's tokens: proj float32 rows [Z | X | G] of `width` columns each;
+        z = sigmoid(Z + z_bias), u = X + x_bias, S <- (1 - z) S + z (u + 1/2 if u >= 0 else sigmoid(u)), per sequence from its state
+        row and back into it.  Returns S silu(G) [T, width] in `out_dtype`.  single: every sequence brings exactly one token."""
+        _need(proj, "proj", torch.float32, 2); _need(state, "state", torch.float32, 2)
+        _need(z_bias, "z_bias", torch.float32, 1); _need(x_bias, "x_bias", torch.float32, 1)
+        T = proj.shape[0]
+        if proj.shape[1] != 3 * width or z_bias.shape[0] != width or x_bias.shape[0] != width or state.shape[1] != width:
+            raise KernelError(f"mingru: rows of {proj.shape[1]}, state rows of {state.shape[1]} for {width} channels")
+        n_seqs = cu_seqlens.shape[0] - 1
+        if single and n_seqs != T:
+            raise KernelError(f"mingru: {T} tokens of {n_seqs} sequences are not one token each")
+        out = torch.empty((T, width), dtype=out_dtype, device=proj.device)
+        st = self._lib("mingru.cu").rv_mingru(
+            _ptr(proj), c_int(proj.shape[1]), _ptr(z_bias), _ptr(x_bias), _ptr(cu_seqlens), _ptr(state_slots), _ptr(state),
+            ctypes.c_longlong(state.stride(0)), _ptr(out), c_int(_DT[out_dtype]), c_int(n_seqs), c_int(width), c_int(1 if single else 0),
+            self._stream())
+        _check("mingru", st)
+        return out
+
+    def bigram_add(self, x, table, token_ids, positions, token_seq, cu_seqlens, state_slots, state, mul_prev: int, mul_cur: int,
+                   buckets: int) -> torch.Tensor:
+        """x + table[row] as float32: row = (previous token * mul_prev + token * mul_cur) mod buckets, and row `buckets` for position
+        0.  The previous token of a sequence's first token in the step is read from its state row (int32 [slots, 1]), and the
+        sequence's last token is left there."""
+        _need(x, "x", dims=2); _need(table, "table", dims=2); _need(token_ids, "token_ids", torch.int32, 1)
+        _need(state, "state", torch.int32, 2)
+        T, cols = x.shape
+        if tuple(table.shape) != (buckets + 1, cols) or token_ids.shape[0] != T:
+            raise KernelError(f"bigram_add: table {tuple(table.shape)} of {buckets} + 1 rows for {token_ids.shape[0]} tokens of {tuple(x.shape)}")
+        out = torch.empty((T, cols), dtype=torch.float32, device=x.device)
+        st = self._lib("streamops.cu").rv_bigram_add(
+            _ptr(x), c_int(self._dt(x, "x")), _ptr(table), c_int(self._dt(table, "table")), _ptr(token_ids), _ptr(positions), _ptr(token_seq),
+            _ptr(cu_seqlens), _ptr(state_slots), _ptr(state), c_int(state.stride(0)), ctypes.c_longlong(mul_prev % buckets),
+            ctypes.c_longlong(mul_cur % buckets), c_int(buckets), _ptr(out), c_int(T), c_int(cols), self._stream())
+        _check("bigram_add", st)
+        return out
 
     def mlstm_scan(self, proj, i_col0: int, f_col0: int, i_bias, f_bias, cu_seqlens, state_slots, state, heads: int, head_dim: int,
                    value_dim: int, cap: float):

@@ -25,12 +25,7 @@ class _Layer:
         self.parts: Dict[str, object] = {}
         self.mixer = None                  # the part that owns the run entry's cache slot, if the layer has one
         for role, ps in spec.parts.items():
-            params = dict(ps.params)
-            if ps.family == "mixer" and "position" in params:
-                key = params["position"]
-                if key is not None and key not in position_encodings:
-                    raise ConfigError(f"layer {spec.prefix!r} names position encoding {key!r}, which the model does not define")
-                params["position"] = position_encodings.get(key) if key is not None else None
+            params = self._with_positions(ps.params, position_encodings) if ps.family == "mixer" else dict(ps.params)
             if ps.family not in FAMILIES:
                 raise ConfigError(f"layer {spec.prefix!r}: part {role!r} has family {ps.family!r} (known: {', '.join(FAMILIES)})")
             part = FAMILIES[ps.family].build(ps.kind, **params)
@@ -38,6 +33,21 @@ class _Layer:
             if ps.family == "mixer":
                 self.mixer = part
         self.block = BLOCKS.build(spec.block.kind, parts=self.parts, **spec.block.params)
+
+    def _with_positions(self, given, position_encodings) -> dict:
+        """A mixer's parameters with the encodings that `position` and `value_position` name in place of the names; the
+        members (`branches`) of a mixer made of mixers are handled alike."""
+        params = dict(given)
+        for role in ("position", "value_position"):
+            key = params.get(role)
+            if key is None:
+                continue
+            if key not in position_encodings:
+                raise ConfigError(f"layer {self.spec.prefix!r} names position encoding {key!r}, which the model does not define")
+            params[role] = position_encodings[key]
+        if "branches" in params:
+            params["branches"] = [dict(b, params=self._with_positions(b.get("params", {}), position_encodings)) for b in params["branches"]]
+        return params
 
     def cache_need(self):
         return self.mixer.cache_need() if self.mixer is not None else None
@@ -61,6 +71,10 @@ class DecoderModel:
         self.logit_hooks = [HOOKS.build(h.kind, **h.params) for h in spec.logit_hooks]
         # hooks on the stream in front of a run entry (what a model adds at the start of a repeated pass)
         self.entry_hooks = [[HOOKS.build(h.kind, **h.params) for h in e.before] for e in spec.run_order]
+        # a hook on the embedded tokens that keeps something per sequence has a cache slot behind those of the run order
+        free = 1 + max((e.cache for e in spec.run_order), default=-1)
+        stateful = [i for i, h in enumerate(self.embedding_hooks) if hasattr(h, "cache_need")]
+        self.hook_slots: Dict[int, int] = {i: free + n for n, i in enumerate(stateful)}
         self.keeps_embedding_output = any(getattr(h, "needs_embedding_output", False) for hs in self.entry_hooks for h in hs)
         self.embedding: Optional[torch.Tensor] = None
         self.lm_head: Optional[torch.Tensor] = None
@@ -124,6 +138,8 @@ class DecoderModel:
                 if need != needs.get(e.cache):
                     raise ConfigError(f"layer {e.layer} reads cache slot {e.cache} but needs {need}, "
                                       f"while its writer provides {needs.get(e.cache)}")
+        for i, slot in self.hook_slots.items():
+            needs[slot] = self.embedding_hooks[i].cache_need()
         return needs
 
     # ---- the forward pass of one step ----------------------------------------------------------
@@ -133,17 +149,22 @@ class DecoderModel:
             x = x.to(self.dtype)       # a table the checkpoint keeps in 32 bits; activations have the engine's type
         for pe in self.position_encodings.values():
             x = pe.on_embeddings(x, ctx)
-        for hook in self.embedding_hooks:
-            x = hook(x, ctx)
+        for i, hook in enumerate(self.embedding_hooks):
+            x = hook(x, ctx, caches.view(self.hook_slots[i])) if i in self.hook_slots else hook(x, ctx)
         ctx.extras["activation_dtype"] = self.dtype
         if self.spec.residual_dtype == "float32" and x.dtype != torch.float32:
             x = x.float()              # the stream between the layers stays in 32 bits; blocks round a copy for their products
         if self.keeps_embedding_output:
             # blocks add into the stream in place: what the embedding section left is kept as a copy
             ctx.extras["embedding_output"] = x.clone()
-        for e, hooks in zip(self.spec.run_order, self.entry_hooks):
+        order = self.spec.run_order
+        for n, (e, hooks) in enumerate(zip(order, self.entry_hooks)):
             for hook in hooks:
                 x = hook(x, ctx)
+            ctx.following_norms = None
+            if n + 1 < len(order) and not self.entry_hooks[n + 1]:
+                offer = getattr(self.layers[order[n + 1].layer].block, "input_norms", None)
+                ctx.following_norms = offer() if offer is not None else None
             x = self.layers[e.layer].block(x, ctx, caches.view(e.cache), e.writes_cache)
         return x
 

@@ -14,8 +14,11 @@ tensors it owns (`tensor_specs`, names relative to its prefix) and receives them
   `CacheView` of the run entry's cache slot (with one sub-view per member of a `CompositeNeed`).
 * feed-forward: `__call__(x, ctx, residual)` -> residual + f(x).
 * block: built from `parts`, the layer's built parts by role name (which roles it needs is the
-  block's own matter), plus its parameters; `__call__(x, ctx, cache, write_cache)` -> x.
-* hook: `__call__(x, ctx)` -> x, on the embedded tokens or on the float32 logits.
+  block's own matter), plus its parameters; `__call__(x, ctx, cache, write_cache)` -> x.  A block whose input is the
+  stream under RMSNorms may offer `input_norms()` -> [(gamma, eps), ...]: the block that runs before it can then form them in the
+  kernel that writes the stream (`ctx.following_norms`, None where something else stands between).
+* hook: `__call__(x, ctx)` -> x, on the embedded tokens or on the float32 logits.  A hook on the embedded tokens that
+  keeps something per sequence offers `cache_need()`; it is then called `(x, ctx, cache)` with a cache slot of its own.
 
 A part whose step cannot be recorded into a CUDA graph (it reads device values on the host, or
 launches a number of kernels that depends on the data) sets `graph_safe = False`; a model with

@@ -202,3 +202,64 @@ class PreNormStreamResidualBlock:
 
 
 BLOCKS.register("prenorm_stream_residual", PreNormStreamResidualBlock)
+
+
+class SideBySideResidualBlock:
+    """`side_by_side_residual`: x + multiplier * (mixer(norm(x)) + feed_forward(norm'(x))): mixer and feed-forward read the
+    SAME x, each under an RMSNorm of its own.  A layer may have no feed-forward.
+
+    The stream x is float32 whatever the engine's type (`ModelSpec.residual_dtype`).  Both norms come from one statistic of
+    the row; the sublayers return float32 (a mixer made of mixers: one term per member with its factor), and one kernel adds
+    all of them to the stream and, where the next block of the run order offers its `input_norms`, leaves that block's
+    inputs as well.  They travel beside the stream in `ctx.extras`; a block that finds none (the first layer) forms them."""
+    ROLES = ("mixer", "mixer_norm")
+    OPTIONAL = ("feed_forward", "feed_forward_norm")
+    KEY = "normed_stream"
+
+    def __init__(self, parts, multiplier: float = 1.0):
+        from ..errors import ConfigError
+        names = set(parts)
+        if not set(self.ROLES) <= names or not names <= set(self.ROLES + self.OPTIONAL) or \
+                (("feed_forward" in names) != ("feed_forward_norm" in names)):
+            raise ConfigError(f"the side-by-side residual block arranges {', '.join(self.ROLES)} and, together, "
+                              f"{', '.join(self.OPTIONAL)}; got {', '.join(sorted(parts))}")
+        self.mixer, self.mixer_norm = parts["mixer"], parts["mixer_norm"]
+        self.feed_forward, self.feed_forward_norm = parts.get("feed_forward"), parts.get("feed_forward_norm")
+        self.multiplier = float(multiplier)
+        for n in (self.mixer_norm, self.feed_forward_norm):
+            if n is not None and not hasattr(n, "as_rms"):
+                raise ConfigError("the side-by-side residual block needs norms that offer `as_rms()` (an RMSNorm)")
+
+    def input_norms(self):
+        return [n.as_rms() for n in (self.mixer_norm, self.feed_forward_norm) if n is not None]
+
+    def __call__(self, x, ctx, cache, write_cache=True):
+        k = ctx.kernels
+        dtype = ctx.extras.get("activation_dtype", x.dtype)
+        if x.dtype != torch.float32:
+            x = x.float()
+        kept = ctx.extras.pop(self.KEY, None)
+        if kept is not None and kept[0] is x:
+            inputs = kept[1]
+        else:
+            inputs = k.stream_combine(x, [], self.input_norms(), dtype)[1]
+        if hasattr(self.mixer, "terms"):
+            terms = self.mixer.terms(inputs[0], ctx, cache, write_cache=write_cache)
+        else:
+            terms = [(self.mixer(inputs[0], ctx, cache, residual=None, write_cache=write_cache, out_dtype=torch.float32), 1.0)]
+        if self.feed_forward is not None:
+            terms.append((self.feed_forward(inputs[1], ctx, residual=None, out_dtype=torch.float32), 1.0))
+        terms = [(y, self.multiplier * c) for y, c in terms]
+        while len(terms) > 3:                        # (the kernel adds three terms at a time)
+            x, _ = k.stream_combine(x, terms[:3], [], dtype)
+            terms = terms[3:]
+        following = ctx.following_norms
+        if following is not None and len(following) > 2:
+            following = None
+        x, normed = k.stream_combine(x, terms, following or [], dtype)
+        if following:
+            ctx.extras[self.KEY] = (x, normed)
+        return x
+
+
+BLOCKS.register("side_by_side_residual", SideBySideResidualBlock)

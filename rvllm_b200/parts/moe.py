@@ -8,7 +8,9 @@ choice is a table lookup by token id.
                  softmax); optionally a shared expert of the same form runs for every token and is added.
                  The experts' matrices are kept stacked ([experts, 2 ff, width] gate rows then up rows, and
                  [experts, width, ff]) so that one kernel serves all of them.
-`routed_moe`     every token runs `top` of `experts` plain MLPs  down_e( act(up_e x) ), act = relu squared, chosen by a router:
+`routed_moe`     every token runs `top` of `experts` MLPs chosen by a router.  An expert is plain, down_e( relu(up_e x)^2 )
+                 ("relu2"), or gated, down_e( silu(gate_e x) * up_e x ) ("silu").  Scoring "softmax": the choice is made among
+                 z = Wr x + correction in float32, the weights are the softmax over the chosen z.  Scoring "sigmoid":
                  s = sigmoid(Wr x) in float32; the choice is made among s + correction (a number per expert), only within
                  the `keep_groups` best of `groups` equal groups of neighbouring experts (a group counts by the sum of its
                  two largest corrected scores); the weights are the chosen experts' s divided by their sum (+ 1e-20).
@@ -96,12 +98,14 @@ class TableMoE(Part):
 
 
 class RoutedMoE(Part):
-    ACTIVATIONS = ("relu2",)
+    ACTIVATIONS = ("relu2", "silu")
+    SCORINGS = ("sigmoid", "softmax")
 
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, groups: int = 1, keep_groups: int = 1,
-                 shared_intermediate_size: Optional[int] = None, activation: str = "relu2", names=("up", "down"),
+                 shared_intermediate_size: Optional[int] = None, activation: str = "relu2", names=None,
                  router: str = "router", correction: str = "correction", expert_prefix: str = "e",
-                 shared_prefix: str = "shared.", shared_gate: str = "sg", suffix: str = "", weight_eps: float = 1e-20):
+                 shared_prefix: str = "shared.", shared_gate: str = "sg", suffix: str = "", weight_eps: float = 1e-20,
+                 scoring: str = "sigmoid"):
         from ..errors import ConfigError
         problems = []
         if not 1 <= top <= experts:
@@ -114,51 +118,73 @@ class RoutedMoE(Part):
             problems.append(f"the router serves at most 1,024 experts, got {experts}")
         if activation not in self.ACTIVATIONS:
             problems.append(f"expert activation {activation!r} is not known ({', '.join(self.ACTIVATIONS)})")
+        if scoring not in self.SCORINGS:
+            problems.append(f"router scoring {scoring!r} is not known ({', '.join(self.SCORINGS)})")
         if problems:
             raise ConfigError(problems, "routed mixture of experts")
         self.hidden_size, self.intermediate_size, self.experts, self.top = hidden_size, intermediate_size, experts, top
         self.groups, self.keep_groups, self.activation, self.weight_eps = groups, keep_groups, activation, weight_eps
-        self.names, self.router_name, self.correction_name, self.expert_prefix = tuple(names), router, correction, expert_prefix
+        self.scoring, self.gated = scoring, activation == "silu"
+        names = tuple(names) if names is not None else (("gate", "up", "down") if self.gated else ("up", "down"))
+        self.names, self.router_name, self.correction_name, self.expert_prefix = names, router, correction, expert_prefix
         self.shared_prefix, self.shared_gate, self.suffix = shared_prefix, shared_gate, suffix
         self.shared_ff = shared_intermediate_size
-        self.shared_up = self.shared_down = None
-        if shared_intermediate_size is not None:
+        self.shared = self.shared_up = self.shared_down = None
+        if shared_intermediate_size is not None and self.gated:
+            self.shared = GatedMLP(hidden_size, shared_intermediate_size, "silu", names=names, suffix=suffix)
+        elif shared_intermediate_size is not None:
             self.shared_up = Linear(hidden_size, [shared_intermediate_size], [names[0]], suffix=suffix)
             self.shared_down = Linear(shared_intermediate_size, [hidden_size], [names[1]], suffix=suffix)
         self.router = self.correction = self.up = self.down = None
 
+    def _shared_parts(self):
+        return [part for part in (self.shared, self.shared_up, self.shared_down) if part is not None]
+
     def tensor_specs(self):
-        u, d = self.names
+        *first, d = self.names                               # (gate and) up, down
         specs = {self.router_name + self.suffix: TensorSpec((self.experts, self.hidden_size), "matrix"),
                  self.correction_name: TensorSpec((self.experts,), "bias")}
         for e in range(self.experts):
             p = f"{self.expert_prefix}{e}."
-            specs[f"{p}{u}{self.suffix}"] = TensorSpec((self.intermediate_size, self.hidden_size), "matrix")
+            for u in first:
+                specs[f"{p}{u}{self.suffix}"] = TensorSpec((self.intermediate_size, self.hidden_size), "matrix")
             specs[f"{p}{d}{self.suffix}"] = TensorSpec((self.hidden_size, self.intermediate_size), "matrix")
-        if self.shared_up is not None:
-            for lin in (self.shared_up, self.shared_down):
-                specs.update({self.shared_prefix + n: ts for n, ts in lin.tensor_specs().items()})
+        if self.shared_ff is not None:
+            for part in self._shared_parts():
+                specs.update({self.shared_prefix + n: ts for n, ts in part.tensor_specs().items()})
             specs[self.shared_prefix + self.shared_gate + self.suffix] = TensorSpec((1, self.hidden_size), "matrix")
         return specs
 
     def bind(self, get):
-        u, d = self.names
+        *first, d = self.names
         rows = [get(self.router_name + self.suffix)]
-        if self.shared_up is not None:                       # the shared expert's gate is one more row of the router's product
+        if self.shared_ff is not None:                       # the shared expert's gate is one more row of the router's product
             rows.append(get(self.shared_prefix + self.shared_gate + self.suffix))
-            self.shared_up.bind(lambda name: get(self.shared_prefix + name))
-            self.shared_down.bind(lambda name: get(self.shared_prefix + name))
+            for part in self._shared_parts():
+                part.bind(lambda name: get(self.shared_prefix + name))
         self.router = torch.cat(rows, dim=0).contiguous()
         self.correction = get(self.correction_name).float().contiguous()       # the router is float32
-        self.up = torch.stack([get(f"{self.expert_prefix}{e}.{u}{self.suffix}") for e in range(self.experts)]).contiguous()
+        # [experts, ff, width], gated experts: [experts, 2 ff, width], an expert's gate rows and then its up rows
+        self.up = torch.stack([torch.cat([get(f"{self.expert_prefix}{e}.{u}{self.suffix}") for u in first], dim=0)
+                               for e in range(self.experts)]).contiguous()
         self.down = torch.stack([get(f"{self.expert_prefix}{e}.{d}{self.suffix}") for e in range(self.experts)]).contiguous()
 
     def __call__(self, x, ctx, residual=None, out_dtype=None):
         k = ctx.kernels
         scores = k.linear(x, self.router, None, None, torch.float32)
         chosen, weights, shared_gate = k.moe_route_top(scores, self.correction, self.experts, self.top, self.groups,
-                                                       self.keep_groups, self.weight_eps, shared_gate=self.shared_up is not None)
+                                                       self.keep_groups, self.weight_eps, shared_gate=self.shared_ff is not None,
+                                                       scoring=self.scoring)
+        if self.shared is not None and residual is None:     # the shared expert's gate is a factor on what the experts' sum adds
+            add = self.shared(x, ctx, out_dtype=torch.float32)
+            return k.moe_experts(x, chosen, self.up, self.down, 1.0, add=add, out_dtype=out_dtype or x.dtype, weights=weights,
+                                 activation=self.activation, add_scale=shared_gate)
         add = residual
+        if self.shared is not None:
+            add = k.moe_experts(x, chosen, self.up, self.down, 1.0, add=self.shared(x, ctx, out_dtype=torch.float32),
+                                out_dtype=torch.float32, weights=weights, activation=self.activation, add_scale=shared_gate)
+            add = k.scaled_sum(add, 1.0, residual if residual.dtype == torch.float32 else residual.float(), 1.0)
+            return add if out_dtype == torch.float32 else add.to(out_dtype or x.dtype)
         if self.shared_up is not None:
             u = self.shared_up(x, ctx, out_dtype=torch.float32)
             a = k.act_rows(u, self.activation, x.dtype, row_scale=shared_gate)      # W (g a) = g (W a): the gate rides on the activation

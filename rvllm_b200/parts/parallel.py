@@ -5,6 +5,8 @@
 `branches` lists the members: {"kind": registry key, "params": {...}, "prefix": tensor sub-prefix, "scale": number}.
 Every member keeps its own cache or state: the part's need is a `CompositeNeed` with one entry per member, and the
 run entry's cache view carries one sub-view per member.  The members return float32 and the sum is float32.
+A block that adds into a float32 stream may ask for the `terms` [(mixer_b(h), scale_b), ...] and form the sum itself.
+A member's `position` / `value_position` names a position encoding of the model, as a mixer's own does.
 """
 from __future__ import annotations
 
@@ -14,7 +16,7 @@ from .base import MIXERS, CompositeNeed, Part
 
 
 class ParallelMixers(Part):
-    def __init__(self, branches, position=None):
+    def __init__(self, branches):
         from ..errors import ConfigError
         if not branches:
             raise ConfigError("a parallel mixer needs at least one member")
@@ -41,11 +43,15 @@ class ParallelMixers(Part):
     def cache_need(self):
         return CompositeNeed(tuple(m.cache_need() for m in self.members))
 
+    def terms(self, x, ctx, cache, write_cache=True):
+        """[(float32 result, factor), ...], one per member, in their order."""
+        return [(m(x, ctx, view, residual=None, write_cache=write_cache, out_dtype=torch.float32), scale)
+                for m, view, scale in zip(self.members, cache.parts, self.scales)]
+
     def __call__(self, x, ctx, cache, residual=None, write_cache=True, out_dtype=None):
         k = ctx.kernels
         total = None
-        for m, view, scale in zip(self.members, cache.parts, self.scales):
-            y = m(x, ctx, view, residual=None, write_cache=write_cache, out_dtype=torch.float32)
+        for y, scale in self.terms(x, ctx, cache, write_cache):
             total = k.scaled_sum(total, 1.0, y, scale)
         if residual is not None:
             total = k.scaled_sum(total, 1.0, residual if residual.dtype == torch.float32 else residual.float(), 1.0)

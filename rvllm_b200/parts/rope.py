@@ -8,6 +8,11 @@ Frequencies are computed in float64 and kept as float32; angles position * inv_f
 their cos/sin are computed in float64 and the tables kept as float32 (the reference rounds
 them to half precision, which this engine does not).  Pairs are (i, i + head_dim/2)
 (v3/crates/rvllm-fused/src/reference.rs:177-203).
+
+The YaRN rule (Peng et al., "YaRN: Efficient Context Window Extension of Large Language Models"): the pair that turns t times
+over the original length L is i(t) = dims ln(L / (2 pi t)) / (2 ln theta); pairs below i(fast) keep their frequency, pairs
+above i(slow) have it divided by `factor`, a linear ramp blends the two between; cos and sin are multiplied by
+0.1 ln(factor) + 1.
 """
 from __future__ import annotations
 
@@ -33,9 +38,26 @@ def inverse_frequencies(head_dim: int, theta: float, scaling: Optional[dict]) ->
             smooth = (orig / wavelen - low) / (high - low)
             blended = (1.0 - smooth) * inv / factor + smooth * inv
             inv = torch.where(wavelen < orig / high, inv, torch.where(wavelen > orig / low, inv / factor, blended))
+        elif kind == "yarn":
+            factor, orig = float(scaling["factor"]), float(scaling["original"])
+
+            def pair_of(turns: float) -> float:
+                return head_dim * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(float(theta)))
+
+            lo = max(math.floor(pair_of(float(scaling["fast"]))), 0)
+            hi = min(math.ceil(pair_of(float(scaling["slow"]))), head_dim - 1)
+            ramp = ((torch.arange(half, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+            inv = inv / factor * ramp + inv * (1.0 - ramp)
         elif kind != "default":
-            raise ConfigError(f"rotary scaling {kind!r} is not supported (known: default, llama3)")
+            raise ConfigError(f"rotary scaling {kind!r} is not supported (known: default, llama3, yarn)")
     return inv.to(torch.float32)
+
+
+def table_amplitude(scaling: Optional[dict]) -> float:
+    """What cos and sin are multiplied by."""
+    if scaling and scaling.get("rope_type") == "yarn":
+        return 0.1 * math.log(float(scaling["factor"])) + 1.0
+    return 1.0
 
 
 class RotaryEncoding(Part):
@@ -52,6 +74,7 @@ class RotaryEncoding(Part):
             raise ConfigError(f"rotary_dim must be even and in (0, head_dim = {head_dim}], got {rotary_dim}")
         self.head_dim, self.theta, self.scaling, self.rotary_dim = head_dim, theta, scaling, rotary_dim
         self.inv_freq = inverse_frequencies(rotary_dim, theta, scaling)
+        self.amplitude = table_amplitude(scaling)
         self.cos = self.sin = None
 
     def prepare(self, max_len: int, device) -> None:
@@ -62,8 +85,8 @@ class RotaryEncoding(Part):
         for s in range(0, max_len, step):
             pos = torch.arange(s, min(max_len, s + step), dtype=torch.float64)
             ang = pos[:, None] * inv[None, :]
-            cos[s:s + step] = torch.cos(ang).to(torch.float32)
-            sin[s:s + step] = torch.sin(ang).to(torch.float32)
+            cos[s:s + step] = (self.amplitude * torch.cos(ang)).to(torch.float32)
+            sin[s:s + step] = (self.amplitude * torch.sin(ang)).to(torch.float32)
         self.cos, self.sin = cos.to(device), sin.to(device)
 
     def rotation_tables(self):

@@ -125,9 +125,12 @@ class EmulatedKernels:
                 out[t] = o.to(q_row.dtype)
         return out
 
-    def moe_experts(self, x, chosen, gate_up, down, weight, add=None, out_dtype=None, weights=None, activation="silu"):
+    def moe_experts(self, x, chosen, gate_up, down, weight, add=None, out_dtype=None, weights=None, activation="silu",
+                    add_scale=None):
         T, ff = x.shape[0], gate_up.shape[1] // 2
         out = torch.zeros((T, x.shape[1])) if add is None else add.clone().float()
+        if add_scale is not None:
+            out *= add_scale[:, None]
         for t in range(T):
             for j, e in enumerate(chosen[t].tolist()):
                 gu = gate_up[e].float() @ x[t].float()
@@ -158,30 +161,33 @@ class EmulatedKernels:
             a = a * row_scale[:, None]
         return a.to(out_dtype)
 
-    def moe_route_top(self, scores, correction, experts, top, groups, keep, weight_eps, shared_gate=False):
-        s = torch.sigmoid(scores[:, :experts].float())
+    def moe_route_top(self, scores, correction, experts, top, groups, keep, weight_eps, shared_gate=False, scoring="sigmoid"):
+        s = torch.sigmoid(scores[:, :experts].float()) if scoring == "sigmoid" else scores[:, :experts].float()
         c = s + correction
         per = experts // groups
         gs = c.view(-1, groups, per).topk(min(2, per), dim=-1).values.sum(-1)
         kept = gs.topk(keep, dim=-1).indices
         allowed = torch.zeros_like(gs, dtype=torch.bool).scatter_(1, kept, True).repeat_interleave(per, dim=1)
         chosen = c.masked_fill(~allowed, float("-inf")).topk(top, dim=-1).indices
-        w = s.gather(1, chosen)
+        w = s.gather(1, chosen) if scoring == "sigmoid" else torch.softmax(c.gather(1, chosen), -1)
         w = w / (w.sum(-1, keepdim=True) + weight_eps)
         gate = torch.sigmoid(scores[:, experts].float()) if shared_gate else None
         return chosen.to(torch.int32), w, gate
 
-    def qk_unit_prepare(self, proj, eps, positions, cos, sin, slot_mapping, cache_layer, num_heads, num_kv_heads, head_dim,
-                        value_dim, slot_dim, out_dtype, halves=False, with_gate=True, write_kv=True):
+    def qk_prepare(self, proj, positions, cos, sin, slot_mapping, cache_layer, num_heads, num_kv_heads, head_dim, value_dim,
+                   slot_dim, out_dtype, eps=None, halves=False, with_gate=False, write_kv=True, maps=1, bias=None, value_tables=None):
         T = proj.shape[0]
-        x = proj.float()
+        x = proj.float().clone()
+        if bias is not None:
+            x[:, :bias.shape[0]] += bias
         pos = positions.long()
 
-        def turn(v):           # [T, heads, head_dim]
+        def turn(v, cos, sin):           # [T, heads, ..., head_dim]
             if cos is None:
                 return v
             half = cos.shape[1]
-            c, s = cos[pos][:, None, :], sin[pos][:, None, :]
+            shape = (T,) + (1,) * (v.dim() - 2) + (half,)
+            c, s = cos[pos].view(shape), sin[pos].view(shape)
             out = v.clone()
             if halves:
                 a, b = v[..., :half], v[..., half:2 * half]
@@ -191,15 +197,21 @@ class EmulatedKernels:
                 out[..., 0:2 * half:2], out[..., 1:2 * half:2] = a * c - b * s, b * c + a * s
             return out
 
-        unit = lambda v: v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)
-        qw = num_heads * head_dim
-        q = torch.zeros((T, num_heads, slot_dim))
-        q[:, :, :head_dim] = unit(turn(x[:, :qw].view(T, num_heads, head_dim)))
+        def norm(v):
+            return v if eps is None else v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)
+
+        qw = num_heads * maps * head_dim
+        turned = norm(turn(x[:, :qw].view(T, num_heads, maps, head_dim), cos, sin))
+        q = torch.zeros((T, num_heads, maps, slot_dim))
+        for m in range(maps):
+            q[:, :, m, m * head_dim:(m + 1) * head_dim] = turned[:, :, m]
         col = qw
         if write_kv:
-            kw, vw = num_kv_heads * head_dim, num_kv_heads * value_dim
-            k = unit(turn(x[:, col:col + kw].view(T, num_kv_heads, head_dim)))
+            kw, vw = num_kv_heads * maps * head_dim, num_kv_heads * value_dim
+            k = norm(turn(x[:, col:col + kw].view(T, num_kv_heads, maps, head_dim), cos, sin)).reshape(T, num_kv_heads, maps * head_dim)
             v = x[:, col + kw:col + kw + vw].view(T, num_kv_heads, value_dim)
+            if value_tables is not None:
+                v = turn(v, *value_tables)
             col += kw + vw
             ps = cache_layer.shape[3]
             for t, slot in enumerate(slot_mapping.tolist()):
@@ -207,10 +219,68 @@ class EmulatedKernels:
                     continue
                 cache_layer[slot // ps, 0, :, slot % ps, :] = 0
                 cache_layer[slot // ps, 1, :, slot % ps, :] = 0
-                cache_layer[slot // ps, 0, :, slot % ps, :head_dim] = k[t].to(cache_layer.dtype)
+                cache_layer[slot // ps, 0, :, slot % ps, :maps * head_dim] = k[t].to(cache_layer.dtype)
                 cache_layer[slot // ps, 1, :, slot % ps, :value_dim] = v[t].to(cache_layer.dtype)
         gate = torch.sigmoid(x[:, col:col + num_heads]) if with_gate else None
-        return q.view(T, num_heads * slot_dim).to(out_dtype), gate
+        return q.view(T, num_heads * maps * slot_dim).to(out_dtype), gate
+
+    def qk_unit_prepare(self, proj, eps, positions, cos, sin, slot_mapping, cache_layer, num_heads, num_kv_heads, head_dim,
+                        value_dim, slot_dim, out_dtype, halves=False, with_gate=True, write_kv=True, value_tables=None):
+        return self.qk_prepare(proj, positions, cos, sin, slot_mapping, cache_layer, num_heads, num_kv_heads, head_dim, value_dim,
+                               slot_dim, out_dtype, eps=eps, halves=halves, with_gate=with_gate, write_kv=write_kv,
+                               value_tables=value_tables)
+
+    def turn_back(self, o, positions, cos, sin, heads, value_dim, slot_dim, halves=True):
+        T, half = o.shape[0], value_dim // 2
+        v = o.view(T, heads, slot_dim)[..., :value_dim].float()
+        c, s = cos[positions.long()][:, None, :], sin[positions.long()][:, None, :]
+        out = torch.empty_like(v)
+        first, second = (slice(0, half), slice(half, value_dim)) if halves else (slice(0, value_dim, 2), slice(1, value_dim, 2))
+        a, b = v[..., first], v[..., second]
+        out[..., first], out[..., second] = a * c + b * s, b * c - a * s
+        return out.reshape(T, heads * value_dim).to(o.dtype)
+
+    def map_difference(self, o, lam, eps, factor, heads, value_dim, slot_dim):
+        T = o.shape[0]
+        v = o.view(T, heads, 2, slot_dim)[..., :value_dim].float()
+        d = v[:, :, 0] - lam * v[:, :, 1]
+        return (factor * d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps)).reshape(T, heads * value_dim).to(o.dtype)
+
+    def stream_combine(self, x, terms, norms, out_dtype):
+        assert len(terms) <= 3 and len(norms) <= 2
+        for y, c in terms:
+            x += c * y
+        return x, [self.rmsnorm(x, gamma, eps).to(out_dtype) for gamma, eps in norms]
+
+    def mingru(self, proj, z_bias, x_bias, cu_seqlens, state_slots, state, width, single, out_dtype):
+        out = torch.zeros((proj.shape[0], width))
+        z = torch.sigmoid(proj[:, :width] + z_bias)
+        u = proj[:, width:2 * width] + x_bias
+        c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+        g = proj[:, 2 * width:]
+        cu = cu_seqlens.tolist()
+        for i, slot in enumerate(state_slots.tolist()):
+            assert not single or cu[i + 1] - cu[i] == 1
+            S = state[slot].clone() if slot >= 0 else torch.zeros(width)
+            for t in range(cu[i], cu[i + 1]):
+                S = (1.0 - z[t]) * S + z[t] * c[t]
+                out[t] = S * g[t] * torch.sigmoid(g[t])
+            if slot >= 0:
+                state[slot] = S
+        return out.to(out_dtype)
+
+    def bigram_add(self, x, table, token_ids, positions, token_seq, cu_seqlens, state_slots, state, mul_prev, mul_cur, buckets):
+        out = x.float().clone()
+        ids, pos, cu = token_ids.tolist(), positions.tolist(), cu_seqlens.tolist()
+        for i, slot in enumerate(state_slots.tolist()):
+            prev = int(state[slot, 0]) if slot >= 0 else 0
+            for t in range(cu[i], cu[i + 1]):
+                row = buckets if pos[t] == 0 else (prev * mul_prev + ids[t] * mul_cur) % buckets
+                out[t] += table[row].float()
+                prev = ids[t]
+            if slot >= 0:
+                state[slot, 0] = prev
+        return out
 
     def mlstm_scan(self, proj, i_col0, f_col0, i_bias, f_bias, cu_seqlens, state_slots, state, heads, head_dim, value_dim, cap):
         T = proj.shape[0]
