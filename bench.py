@@ -2,7 +2,7 @@
 """Benchmark of the engine on one B200: decode tokens per second, prefill, roofline.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers L] [--shape NAME]
-                    [--workload decode|serve|tufirax|vipelix|tibepel|tugodra] [--impl ours|reference]
+                    [--workload decode|serve|tufirax|vipelix|tibepel|tugodra|sozudra] [--impl ours|reference]
 
 The default run has the layer sizes of Llama-3.1-8B (32 layers, hidden 4096, 32 query heads,
 8 key/value heads of 128, MLP 14336, vocabulary 128256, llama3 rotary scaling) with random
@@ -834,11 +834,59 @@ def tugodra_pair(size: dict, vocab: int = 32768):
     return tug, vip
 
 
-def run_tugodra(args):
+def measure_design(cfg_dict, args, gen, PROMPT: int, CTX: int):
+    """({prefill of one prompt, decode of `args.batch` sequences behind such prompts}, kernel library) of a design with random
+    weights, through the step function; decode steps from CUDA graphs unless --eager."""
     import torch
 
     from rvllm_b200 import LLM, config_from_dict
     from rvllm_b200.engine import StepEntry
+
+    batch = args.batch
+    config = config_from_dict(cfg_dict)
+    llm = LLM(config=config, random_weights=True, seed=0, dtype="bfloat16", block_size=16, num_blocks=batch * (CTX // 16) + 8,
+              max_model_len=CTX, max_num_seqs=batch, max_num_batched_tokens=PROMPT, enforce_eager=args.eager)
+    runner, V = llm.engine.runner, llm.engine.spec.vocab_size
+    p = torch.randint(0, V, (PROMPT,), generator=gen).tolist()
+    for _ in range(3):
+        runner.step([StepEntry("w", p, [PROMPT - 1])])
+        runner.finish("w")
+    torch.cuda.synchronize()
+    pf = []
+    for _ in range(3):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        runner.step([StepEntry("p", p, [PROMPT - 1])])
+        b.record()
+        torch.cuda.synchronize()
+        runner.finish("p")
+        pf.append(a.elapsed_time(b))
+    ids = [f"d{i}" for i in range(batch)]
+    for rid in ids:
+        runner.step([StepEntry(rid, torch.randint(0, V, (PROMPT,), generator=gen).tolist(), [])])
+    for _ in range(args.warmup):
+        runner.step([StepEntry(r, [1], [0]) for r in ids])
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(args.steps):
+        runner.step([StepEntry(r, [1], [0]) for r in ids])
+    b.record()
+    torch.cuda.synchronize()
+    ms = a.elapsed_time(b) / args.steps
+    for rid in ids:
+        runner.finish(rid)
+    kernels = llm.engine.kernels
+    kernels.raise_on_abort()
+    del llm
+    torch.cuda.empty_cache()
+    return {"prefill_ms": round(min(pf), 3), "prefill_tok_s": round(PROMPT / (min(pf) / 1e3), 1),
+            "decode_ms_per_step": round(ms, 4), "decode_tok_s": round(batch / (ms / 1e3), 1)}, kernels
+
+
+def run_tugodra(args):
+    import torch
+
     from rvllm_b200.kernels import AttentionMeta
 
     peaks = measured_peaks()
@@ -847,52 +895,11 @@ def run_tugodra(args):
     out = {"workload": "tugodra", "dtype": "bf16", "data": "synthetic", "peaks": peaks["source"], "prompt_len": PROMPT, "batch": batch,
            "steps": args.steps, "warmup": args.warmup, "models": {}, "kernels": {}}
 
-    def measure(cfg_dict):
-        config = config_from_dict(cfg_dict)
-        llm = LLM(config=config, random_weights=True, seed=0, dtype="bfloat16", block_size=16, num_blocks=batch * (CTX // 16) + 8,
-                  max_model_len=CTX, max_num_seqs=batch, max_num_batched_tokens=PROMPT, enforce_eager=args.eager)
-        runner, V = llm.engine.runner, llm.engine.spec.vocab_size
-        p = torch.randint(0, V, (PROMPT,), generator=gen).tolist()
-        for _ in range(3):
-            runner.step([StepEntry("w", p, [PROMPT - 1])])
-            runner.finish("w")
-        torch.cuda.synchronize()
-        pf = []
-        for _ in range(3):
-            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            a.record()
-            runner.step([StepEntry("p", p, [PROMPT - 1])])
-            b.record()
-            torch.cuda.synchronize()
-            runner.finish("p")
-            pf.append(a.elapsed_time(b))
-        ids = [f"d{i}" for i in range(batch)]
-        for rid in ids:
-            runner.step([StepEntry(rid, torch.randint(0, V, (PROMPT,), generator=gen).tolist(), [])])
-        for _ in range(args.warmup):
-            runner.step([StepEntry(r, [1], [0]) for r in ids])
-        torch.cuda.synchronize()
-        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        a.record()
-        for _ in range(args.steps):
-            runner.step([StepEntry(r, [1], [0]) for r in ids])
-        b.record()
-        torch.cuda.synchronize()
-        ms = a.elapsed_time(b) / args.steps
-        for rid in ids:
-            runner.finish(rid)
-        kernels = llm.engine.kernels
-        kernels.raise_on_abort()
-        del llm
-        torch.cuda.empty_cache()
-        return {"prefill_ms": round(min(pf), 3), "prefill_tok_s": round(PROMPT / (min(pf) / 1e3), 1),
-                "decode_ms_per_step": round(ms, 4), "decode_tok_s": round(batch / (ms / 1e3), 1)}, kernels
-
     K = None
     for name in (args.sizes.split(",") if args.sizes else list(TUGODRA_SIZES)):
         tug, vip = tugodra_pair(TUGODRA_SIZES[name])
-        a, K = measure(tug)
-        b, K = measure(vip)
+        a, K = measure_design(tug, args, gen, PROMPT, CTX)
+        b, K = measure_design(vip, args, gen, PROMPT, CTX)
         out["models"][name] = {"tugodra": a, "vipelix_same_size": b, "layers": TUGODRA_SIZES[name]["layers"],
                                "prefill_ratio": round(a["prefill_tok_s"] / b["prefill_tok_s"], 3),
                                "decode_ratio": round(a["decode_tok_s"] / b["decode_tok_s"], 3)}
@@ -1072,6 +1079,194 @@ def run_tugodra(args):
     ms_like = _time_kernel(lambda: K.silu_mul(gub), flush=flush)
     by_bytes("act_rows", _time_kernel(lambda: K.act_rows(u, "relu2", bf, row_scale=sg), flush=flush), T * SF * 6,
              like_bytes("silu_mul", ms_like, T * SF * 6))
+    K.raise_on_abort()
+    print(json.dumps(out))
+
+
+# ---------------------------------------------------------------------------------------------------------
+# --workload sozudra: the Sozudra design (layers of a capped window attention with turned values beside a minGRU, and of a
+# differential attention, each beside routed gated experts with a gated shared one; bigram rows; a float32 stream) at layer
+# sizes that resemble real models, beside the Tugodra decoder of this engine - the closest design: window attention on
+# unit-norm queries and keys, a recurrence, routed experts with a gated shared one, a float32 stream - at the same width, depth,
+# heads, window and experts; then each of the design's own kernels alone beside the like kernel of the engine's other designs,
+# with its bytes or FLOPs over its time against the measured copy bandwidth or bf16 peak.  Random weights; its own JSON line.
+SOZUDRA_SIZES = {
+    "2k": dict(width=2048, heads=16, kv=4, dim=128, window=1024, gru=2048, d_dim=64, d_vdim=128, m_heads=8, m_dim=128, m_vdim=256,
+               e_ff=1408, experts=16, top=2, shared=2816, layers=8),
+    "4k": dict(width=4096, heads=32, kv=8, dim=128, window=1024, gru=4096, d_dim=64, d_vdim=128, m_heads=16, m_dim=128, m_vdim=256,
+               e_ff=2048, experts=32, top=4, shared=4096, layers=8),
+}
+
+
+def sozudra_pair(size: dict, vocab: int = 32768):
+    """(Sozudra configuration, Tugodra configuration): layers with two mixers side by side and layers of differential attention in
+    turn, each with experts; beside as many Tugodra layers of a matrix memory and of window attention in turn."""
+    router = {"experts": size["experts"], "top": size["top"]}
+    mlp = {"kind": "moe", "expert": {"ff": size["e_ff"]}, "router": router, "shared": {"ff": size["shared"]}}
+    rot = lambda dims: {"dims": dims, "base": 1e6, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}
+    left = {"heads": size["heads"], "kv_heads": size["kv"], "dim": size["dim"], "vdim": size["dim"], "scale": size["dim"] ** -0.5,
+            "softcap": 30.0, "mask": {"size": size["window"]}, "rot": rot(size["dim"])}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {"left": left, "right": {"width": size["gru"]}, "left_scale": 0.5, "right_scale": 0.9}}
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": size["heads"], "kv_heads": size["kv"], "dim": size["d_dim"], "vdim": size["d_vdim"], "scale": size["d_dim"] ** -0.5,
+                     "softcap": 40.0, "diff": 0.2, "mask": {"size": size["window"]}, "rot": rot(size["d_dim"])}}
+    soz = {"architecture": "Sozudra", "width": size["width"], "vocab": vocab, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+           "embedding": {"bigram": {"buckets": 8191, "mul_prev": 4093, "mul_cur": 17}}, "layers": [par, att] * (size["layers"] // 2)}
+    t_att = {"heads": size["heads"], "kv_heads": size["kv"], "dim": size["dim"], "vdim": size["dim"], "scale": size["dim"] ** 0.5 * 0.1,
+             "mask": {"size": size["window"]}, "rot": {"dims": size["dim"], "base": 1e6}}
+    mem = {"heads": size["m_heads"], "dim": size["m_dim"], "vdim": size["m_vdim"], "gate_cap": 15.0}
+    tug = {"architecture": "Tugodra", "width": size["width"], "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": size["width"] ** 0.5},
+           "layers": [{"type": "mlstm", "mixer": mem, "mlp": mlp}, {"type": "attention", "mixer": t_att, "mlp": mlp}] * (size["layers"] // 2)}
+    return soz, tug
+
+
+def run_sozudra(args):
+    import torch
+
+    from rvllm_b200.kernels import AttentionMeta
+
+    peaks = measured_peaks()
+    PROMPT, CTX, batch = 2048, 4096, args.batch
+    gen = torch.Generator().manual_seed(0)
+    out = {"workload": "sozudra", "dtype": "bf16", "data": "synthetic", "peaks": peaks["source"], "prompt_len": PROMPT, "batch": batch,
+           "steps": args.steps, "warmup": args.warmup, "models": {}, "kernels": {}}
+    K = None
+    for name in (args.sizes.split(",") if args.sizes else list(SOZUDRA_SIZES)):
+        soz, tug = sozudra_pair(SOZUDRA_SIZES[name])
+        a, K = measure_design(soz, args, gen, PROMPT, CTX)
+        b, K = measure_design(tug, args, gen, PROMPT, CTX)
+        out["models"][name] = {"sozudra": a, "tugodra_same_size": b, "layers": SOZUDRA_SIZES[name]["layers"],
+                               "prefill_ratio": round(a["prefill_tok_s"] / b["prefill_tok_s"], 3),
+                               "decode_ratio": round(a["decode_tok_s"] / b["decode_tok_s"], 3)}
+
+    # ---- the design's kernels alone, at the "4k" sizes, beside the like kernel ---------------------------------------
+    torch.manual_seed(0)
+    z = SOZUDRA_SIZES["4k"]
+    dev, bf = "cuda", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    bw, peak = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    timed = lambda fn: _time_kernel(fn, flush=flush)
+
+    def by_bytes(name, fn, nbytes, like_name, like_fn, like_bytes):
+        ms_like, ms = timed(like_fn), timed(fn)
+        frac, lfrac = nbytes / (ms / 1e3) / bw, like_bytes / (ms_like / 1e3) / bw
+        out["kernels"][name] = {"ms": round(ms, 4), "gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(frac, 4), "farther_than_like": round(lfrac / frac, 2),
+                                "like": {"kernel": like_name, "ms": round(ms_like, 4), "frac_hbm": round(lfrac, 4)}}
+
+    def by_flops(name, fn, flops, like_name, like_fn, like_flops):
+        ms_like, ms = timed(like_fn), timed(fn)
+        frac, lfrac = flops / (ms / 1e3) / peak, like_flops / (ms_like / 1e3) / peak
+        out["kernels"][name] = {"ms": round(ms, 4), "tflops": round(flops / ms / 1e9, 1), "frac_bf16": round(frac, 4), "farther_than_like": round(lfrac / frac, 2),
+                                "like": {"kernel": like_name, "ms": round(ms_like, 4), "frac_bf16": round(lfrac, 4)}}
+
+    W, H, G, D, WIN, HD, VD = z["width"], z["heads"], z["kv"], z["dim"], z["window"], z["d_dim"], z["d_vdim"]
+    pages = PROMPT // 16
+    pos = torch.arange(PROMPT, dtype=torch.int32, device=dev)
+    seq0, cu0, slot0 = torch.zeros_like(pos), torch.tensor([0, PROMPT], dtype=torch.int32, device=dev), torch.zeros(1, dtype=torch.int32, device=dev)
+
+    def tables(dims):
+        ang = torch.arange(PROMPT, dtype=torch.float64)[:, None] * torch.tensor([1e6 ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)[None, :]
+        return torch.cos(ang).float().to(dev), torch.sin(ang).float().to(dev)
+
+    # -- the stream and the norms of the next layer; the bigram rows
+    g = torch.ones(W, dtype=bf, device=dev)
+    for label, T in (("prefill", PROMPT), ("decode", batch)):
+        x, y1, y2, y3 = (torch.randn(T, W, device=dev) for _ in range(4))
+        by_bytes(f"stream_combine_{label}", lambda: K.stream_combine(x, [(y1, 0.4), (y2, 0.8), (y3, 0.5)], [(g, 1e-6), (g, 1e-6)], bf), T * W * (8 + 12 + 4),
+                 "residual_rmsnorm with the next norm", lambda: K.residual_rmsnorm(y1, g, 1e-6, x, bf, next_norm=(g, 1e-6)), T * W * 14)
+    xe = torch.randn(PROMPT, W, device=dev).to(bf)
+    table = torch.randn(8192, W, device=dev).to(bf)
+    ids = torch.randint(0, 32768, (PROMPT,), device=dev, dtype=torch.int32)
+    prev = torch.zeros(1, 1, dtype=torch.int32, device=dev)
+    by_bytes("bigram_add", lambda: K.bigram_add(xe, table, ids, pos, seq0, cu0, slot0, prev, 4093, 17, 8191), PROMPT * W * 8,
+             "scale_rows", lambda: K.scale_rows(xe, 3.0), PROMPT * W * 6)
+
+    # -- around the attention kernels
+    cos, sin = tables(D)
+    cos_d, sin_d = tables(HD)
+    cache = torch.zeros(pages, 2, G, 16, D, dtype=bf, device=dev)
+    for label, T in (("prefill", PROMPT), ("decode", batch)):
+        p_ = pos[:T].contiguous()
+        pr_like = torch.randn(T, (H + 2 * G) * D + H, device=dev)
+        pr = pr_like[:, :(H + 2 * G) * D].contiguous()
+        n_like = T * (pr_like.shape[1] * 4 + (H + 2 * G) * D * 2 + H * 4)
+        like = ("qk_unit_prepare with a gate", lambda: K.qk_unit_prepare(pr_like, 1e-6, p_, cos, sin, p_, cache, H, G, D, D, D, bf, halves=True), n_like)
+        by_bytes(f"qk_prepare_turned_values_{label}", lambda: K.qk_unit_prepare(pr, 1e-6, p_, cos, sin, p_, cache, H, G, D, D, D, bf, halves=True, with_gate=False,
+                                                                              value_tables=(cos, sin)), T * pr.shape[1] * 6, *like)
+        pr2 = torch.randn(T, 2 * H * HD + G * (2 * HD + VD), device=dev)
+        bias = torch.randn(pr2.shape[1], device=dev)
+        by_bytes(f"qk_prepare_two_maps_{label}", lambda: K.qk_prepare(pr2, p_, cos_d, sin_d, p_, cache, H, G, HD, VD, D, bf, halves=True, maps=2, bias=bias),
+                 T * (pr2.shape[1] * 4 + (2 * H + 2 * G) * D * 2), *like)
+        o1, o2 = torch.randn(T, H * D, device=dev).to(bf), torch.randn(T, 2 * H * D, device=dev).to(bf)
+        of, gam, zg = torch.randn(T, H * D, device=dev), torch.ones(D, dtype=bf, device=dev), torch.randn(T, H * D, device=dev)
+        like = ("head_norm_gate", lambda: K.head_norm_gate(of, gam, 1e-6, zg, 0, H, D, bf), T * H * D * 10)
+        by_bytes(f"turn_back_{label}", lambda: K.turn_back(o1, p_, cos, sin, H, D, D), T * H * D * 4, *like)
+        by_bytes(f"map_difference_{label}", lambda: K.map_difference(o2, 0.4, 1e-6, 0.7, H, VD, D), T * H * D * 6, *like)
+
+    # -- attention inside a window with a capped score, one map and two, beside the window attention with a gate
+    def paged_case(q_len, ctx, seqs, heads):
+        n = seqs * (ctx // 16)
+        kv = torch.randn(n, 2, G, 16, D, device=dev).to(bf)
+        tbl = torch.arange(n, dtype=torch.int32, device=dev).view(seqs, ctx // 16)
+        cu = torch.arange(seqs + 1, dtype=torch.int32, device=dev) * q_len
+        meta = AttentionMeta(tbl, cu, torch.full((seqs,), ctx, dtype=torch.int32, device=dev),
+                             torch.arange(seqs, dtype=torch.int32, device=dev).repeat_interleave(q_len), None, seqs, q_len, ctx, 16,
+                             seqs if q_len == 1 else 0)
+        return torch.randn(seqs * q_len, heads * D, device=dev).to(bf), kv, meta, torch.rand(seqs * q_len, heads, device=dev)
+
+    seen = sum(min(i + 1, WIN) for i in range(PROMPT))
+    q1, kv, meta, gate = paged_case(PROMPT, PROMPT, 1, H)
+    q2 = torch.randn(PROMPT, 2 * H * D, device=dev).to(bf)
+    like = ("window attention with a gate", lambda: K.paged_attention(q1, kv, meta, H, G, D, 0.09, WIN, gate=gate), 4.0 * H * D * seen)
+    by_flops("window_attention_cap_prefill", lambda: K.paged_attention(q1, kv, meta, H, G, D, 0.09, WIN, softcap=30.0), 4.0 * H * D * seen, *like)
+    # (two maps: q.k over a map's elements counts, its product with the other map's half of the key row does not)
+    by_flops("two_map_attention_prefill", lambda: K.paged_attention(q2, kv, meta, 2 * H, G, D, 0.12, WIN, softcap=40.0), 2.0 * 2 * H * (HD + VD) * seen, *like)
+    d1, kvd, dmeta, dgate = paged_case(1, PROMPT, batch, H)
+    d2 = torch.randn(batch, 2 * H * D, device=dev).to(bf)
+    n_kv = batch * WIN * 2 * G * D * 2
+    like = ("window attention with a gate", lambda: K.paged_attention(d1, kvd, dmeta, H, G, D, 0.09, WIN, gate=dgate), n_kv)
+    by_bytes("window_attention_cap_decode", lambda: K.paged_attention(d1, kvd, dmeta, H, G, D, 0.09, WIN, softcap=30.0), n_kv, *like)
+    by_bytes("two_map_attention_decode", lambda: K.paged_attention(d2, kvd, dmeta, 2 * H, G, D, 0.12, WIN, softcap=40.0), n_kv, *like)
+
+    # -- the recurrence beside the engine's other scan with a state per channel (mamba1, 16 states) and the matrix memory
+    C, N = z["gru"], 16
+    zb, xb = torch.zeros(C, device=dev), torch.zeros(C, device=dev)
+    a_, dskip, dtb = -torch.rand(C, N, device=dev), torch.ones(C, device=dev), torch.zeros(C, device=dev)
+    MH, MD, MV = z["m_heads"], z["m_dim"], z["m_vdim"]
+    ib, fb, gcol = torch.zeros(MH, device=dev), torch.full((MH,), 3.0, device=dev), 2 * MH * MD + MH * MV
+    for label, q_len, seqs in (("prefill", PROMPT, 1), ("decode", 1, batch)):
+        T = q_len * seqs
+        cu = torch.arange(seqs + 1, dtype=torch.int32, device=dev) * q_len
+        slots = torch.arange(seqs, dtype=torch.int32, device=dev)
+        pr, st = torch.randn(T, 3 * C, device=dev), torch.zeros(seqs, C, device=dev)
+        u, dtr, bc, zz = torch.randn(T, C, device=dev).to(bf), torch.randn(T, C, device=dev), torch.randn(T, 2 * N, device=dev), torch.randn(T, C, device=dev)
+        st1 = torch.zeros(seqs, C * N, device=dev)
+        by_bytes(f"mingru_{label}", lambda: K.mingru(pr, zb, xb, cu, slots, st, C, q_len == 1, bf), T * C * 14 + seqs * C * 8, "selective_scan",
+                 lambda: K.selective_scan(u, dtr, dtb, a_, bc, 0, N, dskip, zz, 0, cu, slots, st1, bf), T * C * 12 + T * 2 * N * 4 + seqs * C * N * 8)
+        prm, stm = torch.randn(T, gcol + MH * MV + 2 * MH, device=dev), torch.zeros(seqs, MH * MD * (MV + 1) + MH, device=dev)
+        ms = timed(lambda: K.mlstm_scan(prm, gcol + MH * MV, gcol + MH * MV + MH, ib, fb, cu, slots, stm, MH, MD, MV, 15.0))
+        nb = seqs * MH * MD * (MV + 1) * 8 + T * (2 * MH * MD + MH * MV + MH * (MV + 1)) * 4
+        out["kernels"][f"mingru_{label}"]["mlstm_scan"] = {"ms": round(ms, 4), "frac_hbm": round(nb / (ms / 1e3) / bw, 4)}
+
+    # -- the router, and the gated experts beside the squared-relu experts
+    E, top_k, EF = z["experts"], z["top"], z["e_ff"]
+    corr = torch.zeros(E, device=dev)
+    up, gate_up = torch.randn(E, EF, W, device=dev).to(bf) * 0.02, torch.randn(E, 2 * EF, W, device=dev).to(bf) * 0.02
+    down = torch.randn(E, W, EF, device=dev).to(bf) * 0.02
+    for label, T in (("prefill", PROMPT), ("decode", batch)):
+        logits, x, add = torch.randn(T, E + 1, device=dev), torch.randn(T, W, device=dev).to(bf), torch.randn(T, W, device=dev)
+        n = T * ((E + 1) * 4 + top_k * 8 + 4)
+        by_bytes(f"moe_route_top_softmax_{label}", lambda: K.moe_route_top(logits, corr, E, top_k, 1, 1, 0.0, shared_gate=True, scoring="softmax"), n,
+                 "moe_route_top (sigmoid)", lambda: K.moe_route_top(logits, corr, E, top_k, 1, 1, 1e-20, shared_gate=True), n)
+        chosen, wts, sg = K.moe_route_top(logits, corr, E, top_k, 1, 1, 0.0, shared_gate=True, scoring="softmax")
+        gated = lambda: K.moe_experts(x, chosen, gate_up, down, 1.0, add=add, out_dtype=torch.float32, weights=wts, activation="silu", add_scale=sg)
+        plain = lambda: K.moe_experts(x, chosen, up, down, 1.0, add=add, out_dtype=torch.float32, weights=wts, activation="relu2")
+        if label == "prefill":
+            by_flops("gated_experts_prefill", gated, 6.0 * T * top_k * EF * W, "squared-relu experts", plain, 4.0 * T * top_k * EF * W)
+        else:
+            touched = len(set(chosen.flatten().tolist()))
+            by_bytes("gated_experts_decode", gated, touched * 3 * EF * W * 2, "squared-relu experts", plain, touched * 2 * EF * W * 2)
+            out["kernels"]["gated_experts_decode"]["experts_touched"] = touched
     K.raise_on_abort()
     print(json.dumps(out))
 
@@ -1298,10 +1493,10 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the shape has (both numbers are reported)")
     ap.add_argument("--shape", default="llama-3.1-8b", choices=sorted(SHAPES), help="layer sizes of the model")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "tufirax", "vipelix", "tibepel", "tugodra"],
-                    help="decode: the benchmark's one JSON line; serve: continuous batching of uneven prompts; tufirax, vipelix, tibepel: "
-                         "that design at real layer sizes beside the closest decoder of equal size, and its kernels alone")
-    ap.add_argument("--sizes", default="", help="tufirax, vipelix, tibepel, tugodra: which sizes to run, with commas (default: all)")
+    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "tufirax", "vipelix", "tibepel", "tugodra", "sozudra"],
+                    help="decode: the benchmark's one JSON line; serve: continuous batching of uneven prompts; tufirax, vipelix, tibepel, "
+                         "tugodra, sozudra: that design at real layer sizes beside the closest decoder of equal size, and its kernels alone")
+    ap.add_argument("--sizes", default="", help="tufirax, vipelix, tibepel, tugodra, sozudra: which sizes to run, with commas (default: all)")
     ap.add_argument("--requests", type=int, default=64, help="serve: number of requests")
     ap.add_argument("--output-len", type=int, default=256, help="serve: tokens generated per request")
     ap.add_argument("--budget", type=int, default=2048, help="serve: tokens per step")
@@ -1327,6 +1522,8 @@ def main():
         run_tibepel(args)
     elif args.workload == "tugodra":
         run_tugodra(args)
+    elif args.workload == "sozudra":
+        run_sozudra(args)
     elif args.workload == "serve":
         run_serve(args)
     else:

@@ -6,17 +6,20 @@
 // with [Z | X | G] the columns of a float32 projection.  S is kept per request and channel in float32; y is rounded once.
 //
 // A step S -> a S + b is an affine map, and affine maps compose: (a2, b2) after (a1, b1) is (a1 a2, a2 b1 + b2).  So a prompt
-// portion is not walked token by token: a CTA owns 32 channels of one sequence and takes MG_WARPS * MG_RUN tokens at a time.
-// Each warp forms the maps of MG_RUN neighbouring tokens in registers (a lane per channel) and their composition; the
-// compositions go through shared memory, every warp applies those of the warps before it to the state that the tokens so
-// far have left, and then applies its own maps one by one.  The next tokens' inputs are loaded before the exchange and wait
-// in registers.  Steps of single tokens take a kernel with a thread per channel.
+// portion is not walked token by token: a CTA owns MG_CHANNELS channels of one sequence and takes MG_RUNS * MG_RUN tokens at a
+// time.  A thread forms the maps of MG_RUN neighbouring tokens of one channel in registers and their composition; the
+// compositions go through shared memory, every thread applies those of the runs before its own to the state that the tokens
+// so far have left, and then applies its own maps one by one.  The next tokens' inputs are loaded before the exchange and
+// wait in registers.  Sixteen channels a CTA (rows of 64 bytes) leave room for two CTAs on an SM, one of which computes while
+// the other waits for its loads or its barrier.  Steps of single tokens take a kernel with a thread per channel.
 //
 // state [slots][channels]; a sequence with slot -1 starts from zero and leaves no state.  Nothing is read on the host.
 #include "common.cuh"
 
-#define MG_WARPS 16
-#define MG_RUN 8
+#define MG_CHANNELS 16
+#define MG_RUNS 32
+#define MG_RUN 4
+#define MG_THREADS (MG_CHANNELS * MG_RUNS)
 
 __device__ __forceinline__ float mg_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 
@@ -31,16 +34,16 @@ __device__ __forceinline__ void mg_store(void* out, int dtype, size_t i, float v
     else ((__nv_bfloat16*)out)[i] = __float2bfloat16_rn(v);
 }
 
-// grid (channel blocks of 32, sequences)
-__global__ void __launch_bounds__(MG_WARPS * 32)
+// grid (channel blocks, sequences)
+__global__ void __launch_bounds__(MG_THREADS, 2)
 mingru_scan_kernel(const float* __restrict__ proj, int stride, const float* __restrict__ z_bias, const float* __restrict__ x_bias,
                    const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, float* __restrict__ state,
                    long long state_stride, void* __restrict__ out, int out_dtype, int channels) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
-    __shared__ float2 maps[2][MG_WARPS][32];
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int ch = blockIdx.x * 32 + lane, seq = blockIdx.y;
+    __shared__ float2 maps[2][MG_RUNS][MG_CHANNELS];
+    const int lane = threadIdx.x % MG_CHANNELS, run = threadIdx.x / MG_CHANNELS;
+    const int ch = blockIdx.x * MG_CHANNELS + lane, seq = blockIdx.y;
     const bool live = ch < channels;
     const int first = cu_seqlens[seq], end = cu_seqlens[seq + 1];
     const int slot = state_slots[seq];
@@ -58,9 +61,9 @@ mingru_scan_kernel(const float* __restrict__ proj, int stride, const float* __re
             g[i] = in ? __ldg(p + 2 * channels) : 0.f;
         }
     };
-    int t0 = first + warp * MG_RUN;
+    int t0 = first + run * MG_RUN;
     fetch(t0);
-    for (int base = first, turn = 0; base < end; base += MG_WARPS * MG_RUN, turn ^= 1) {
+    for (int base = first, turn = 0; base < end; base += MG_RUNS * MG_RUN, turn ^= 1) {
         float a[MG_RUN], b[MG_RUN], gate[MG_RUN];
         float A = 1.f, B = 0.f;
 #pragma unroll
@@ -72,14 +75,14 @@ mingru_scan_kernel(const float* __restrict__ proj, int stride, const float* __re
             B = fmaf(a[i], B, b[i]);
         }
         const int mine = t0;
-        t0 += MG_WARPS * MG_RUN;
+        t0 += MG_RUNS * MG_RUN;
         fetch(t0);
-        maps[turn][warp][lane] = make_float2(A, B);
-        __syncthreads();                                            // (two places in turn: one barrier a round is enough)
+        maps[turn][run][lane] = make_float2(A, B);
+        __syncthreads();                                            // (two places in turn: one barrier a pass is enough)
         float before = S;
 #pragma unroll
-        for (int w = 0; w < MG_WARPS; ++w) {
-            if (w == warp) before = S;
+        for (int w = 0; w < MG_RUNS; ++w) {
+            if (w == run) before = S;
             const float2 m = maps[turn][w][lane];
             S = fmaf(m.x, S, m.y);
         }
@@ -89,7 +92,7 @@ mingru_scan_kernel(const float* __restrict__ proj, int stride, const float* __re
             if (live && mine + i < end) mg_store(out, out_dtype, (size_t)(mine + i) * channels + ch, before * gate[i]);
         }
     }
-    if (warp == 0 && live && slot >= 0 && end > first) state[(size_t)slot * state_stride + ch] = S;
+    if (run == 0 && live && slot >= 0 && end > first) state[(size_t)slot * state_stride + ch] = S;
 }
 
 // one token per sequence; grid (channel blocks, sequences)
@@ -123,7 +126,7 @@ RV_EXPORT int rv_mingru(const float* proj, int stride, const float* z_bias, cons
         RV_LAUNCH_ST = rv_launch(mingru_token_kernel, dim3((channels + 127) / 128, n_seqs), dim3(128), 0, stream, proj, stride, z_bias,
                                  x_bias, state_slots, state, state_stride, out, out_dtype, channels);
     else
-        RV_LAUNCH_ST = rv_launch(mingru_scan_kernel, dim3((channels + 31) / 32, n_seqs), dim3(MG_WARPS * 32), 0, stream, proj, stride,
+        RV_LAUNCH_ST = rv_launch(mingru_scan_kernel, dim3((channels + MG_CHANNELS - 1) / MG_CHANNELS, n_seqs), dim3(MG_THREADS), 0, stream, proj, stride,
                                  z_bias, x_bias, cu_seqlens, state_slots, state, state_stride, out, out_dtype, channels);
     return rv_launch_status();
 }

@@ -231,7 +231,7 @@ def gru_weights(width, n_in, seed=0):
 @BOTH
 @pytest.mark.parametrize("width", [1, 33, 96, 130, 512])
 def test_min_gru_in_portions_against_the_whole_sequence(K, dtype, width):
-    """Portions shorter and longer than a round of the scan (128 tokens), ending inside and at its edges, beside single
+    """Portions shorter and longer than a pass of the scan (128 tokens), ending inside and at its edges, beside single
     tokens of other sequences; a sequence in no slot; a slot nobody holds stays as it is."""
     w = gru_weights(width, 12, seed=width)
     hs = [rnd(n, 12, seed=n).float().double() for n in (301, 140, 5)]
