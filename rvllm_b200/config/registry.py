@@ -15,6 +15,7 @@ from .vipelix_config import VipelixConfig
 from .tibepel_config import TibepelConfig
 from .tugodra_config import TugodraConfig
 from .sozudra_config import SozudraConfig
+from .lefolorn_config import LefolornConfig
 
 _ARCHITECTURES: Dict[str, Type] = {}
 
@@ -61,3 +62,4 @@ register_architecture("Vipelix", VipelixConfig)
 register_architecture("Tibepel", TibepelConfig)
 register_architecture("Tugodra", TugodraConfig)
 register_architecture("Sozudra", SozudraConfig)
+register_architecture("Lefolorn", LefolornConfig)

@@ -29,19 +29,12 @@ from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional, Tuple
 
 from ..errors import ConfigError
+from .reader import NumberReader, is_int
 from .spec import LayerSpec, ModelSpec, PartSpec, RunEntry
 
 DEFAULT_MAX_POSITIONS = 1 << 17       # the design sets no limit; the engine's tables are built for max_model_len
 MIXERS = ("parallel", "attention")
 SCALING = ("factor", "original", "fast", "slow")
-
-
-def _is_int(v) -> bool:
-    return isinstance(v, int) and not isinstance(v, bool)
-
-
-def _is_num(v) -> bool:
-    return isinstance(v, (int, float)) and not isinstance(v, bool)
 
 
 @dataclass(frozen=True)
@@ -51,25 +44,8 @@ class SozudraLayer:
     mlp: Optional[Dict[str, Any]]          # None | {ff, experts, top, shared_ff | None}
 
 
-class _Reader:
-    """Reads numbers out of nested objects and collects what is wrong with them."""
-
-    def __init__(self):
-        self.problems: List[str] = []
-
-    def integer(self, d, key, what, minimum=1):
-        v = d.get(key) if isinstance(d, dict) else None
-        if not _is_int(v) or v < minimum:
-            self.problems.append(f"{what}`{key}` must be an integer >= {minimum}, got {v!r}")
-            return max(minimum, 1)
-        return v
-
-    def number(self, d, key, what, positive=True):
-        v = d.get(key) if isinstance(d, dict) else None
-        if not _is_num(v) or (positive and not v > 0):
-            self.problems.append(f"{what}`{key}` must be a number{' > 0' if positive else ''}, got {v!r}")
-            return 1.0
-        return float(v)
+class _Reader(NumberReader):
+    """... and this design's mixers and feed-forwards."""
 
     def attention(self, m, at: str, differential: bool) -> Dict[str, Any]:
         if not isinstance(m, dict):
@@ -193,14 +169,14 @@ class SozudraConfig:
                 p.append(f"loop: start {start} and stop {stop} must name a span of the {len(raw_layers)} layers")
             loop = (start, stop, times)
         max_pos = obj.get("max_positions", DEFAULT_MAX_POSITIONS)
-        if not _is_int(max_pos) or max_pos < 1:
+        if not is_int(max_pos) or max_pos < 1:
             p.append(f"`max_positions` must be a positive integer, got {max_pos!r}")
             max_pos = DEFAULT_MAX_POSITIONS
         eos = obj.get("eos_token_id")
         eos_ids: Tuple[int, ...] = ()
-        if _is_int(eos):
+        if is_int(eos):
             eos_ids = (eos,)
-        elif isinstance(eos, list) and all(_is_int(t) for t in eos):
+        elif isinstance(eos, list) and all(is_int(t) for t in eos):
             eos_ids = tuple(eos)
         elif eos is not None:
             p.append(f"`eos_token_id` must be an integer or a list of integers, got {eos!r}")

@@ -97,7 +97,15 @@ struct FlashParams {
     float scale_over_cap;          // scale / c
     const float* sinks;            // [nh] or null
     const float* gate;             // [n_tokens, nh] or null
+    // ... and a bias per (distance, head) in units of log2, [nkv][dist_n][nh / nkv]; a distance beyond the last reads the last
+    const float* dist;             // or null
+    int dist_n;
 };
+
+// What the bias adds to the score of a row of head `in_group` of kv head `kvh` (of G heads), `distance` >= 0 positions back.
+__device__ __forceinline__ float flash_distance(const FlashParams& p, int kvh, int in_group, int G, int distance) {
+    return __ldg(p.dist + ((size_t)kvh * p.dist_n + min(distance, p.dist_n - 1)) * G + in_group);
+}
 
 // The score in units of log2: scale * raw, or with a cap c: c * tanh(scale * raw / c) (tanh as 1 - 2 / (e^2x + 1)).
 __device__ __forceinline__ float flash_score(float raw, const FlashParams& p) {
@@ -122,7 +130,8 @@ __device__ __forceinline__ float flash_final(float m, float l, const float* sink
     return inv;
 }
 
-template <int WARPS_M, int WARPS_N, int NSTAGES>
+// DIST: the build with a distance bias (the lookups cost registers, which the others keep for occupancy)
+template <int WARPS_M, int WARPS_N, int NSTAGES, bool DIST>
 __global__ void __launch_bounds__(WARPS_M * WARPS_N * 32)
 flash_paged_kernel(const FlashParams p) {
     rv_pdl_launch_dependents();
@@ -272,7 +281,8 @@ flash_paged_kernel(const FlashParams p) {
                 const int i = e >> 1;
                 const int key = key0 + n * 8 + (e & 1);
                 const bool see = key <= pos[i] && key >= lo[i];
-                const float v = see ? flash_score(s[n][e], p) : -INFINITY;
+                float v = see ? flash_score(s[n][e], p) : -INFINITY;
+                if (DIST && see) v += flash_distance(p, kvh, head[i] - kvh * G, G, pos[i] - key);
                 s[n][e] = v;
                 m_tile[i] = fmaxf(m_tile[i], v);
             }
@@ -530,7 +540,7 @@ __device__ __forceinline__ int tma_swz(int row, int col) {
 }
 __device__ __forceinline__ void consumer_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-template <int NST>
+template <int NST, bool DIST>
 __global__ void __launch_bounds__(TMA_THREADS, TMA_MIN_CTAS)
 flash_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FlashParams p, int* status, int early) {
     rv_pdl_launch_dependents();
@@ -690,7 +700,8 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FlashP
                     const int i = e >> 1;
                     const int key = key0 + n * 8 + (e & 1);
                     const bool see = key <= pos[i] && key >= lo[i];
-                    const float v = see ? flash_score(s[n][e], p) : -INFINITY;
+                    float v = see ? flash_score(s[n][e], p) : -INFINITY;
+                    if (DIST && see) v += flash_distance(p, kvh, head[i] - kvh * G, G, pos[i] - key);
                     s[n][e] = v;
                     m_tile[i] = fmaxf(m_tile[i], v);
                 }
@@ -1487,14 +1498,14 @@ RV_EXPORT int rv_flash_decode_balanced(const void* q, const void* cache, const i
     return rv_launch_status();
 }
 
-template <int WARPS_M, int WARPS_N, int NSTAGES>
+template <int WARPS_M, int WARPS_N, int NSTAGES, bool DIST = false>
 static int launch_flash(const FlashParams& p, int num_seqs, cudaStream_t stream) {
     const int merge_bytes = WARPS_N > 1 ? WARPS_N * 16 * (V_DIM + 2) * 4 : 0;
     const int smem = max(NSTAGES * STAGE_TILES * TILE_BYTES, merge_bytes);
     static RvPerDevice configured;
-    if (int e = rv_configure_smem(configured, flash_paged_kernel<WARPS_M, WARPS_N, NSTAGES>, smem)) return e;
+    if (int e = rv_configure_smem(configured, flash_paged_kernel<WARPS_M, WARPS_N, NSTAGES, DIST>, smem)) return e;
     const dim3 grid(p.row_tiles * p.num_splits, p.nkv, num_seqs);
-    RV_LAUNCH_ST = rv_launch(flash_paged_kernel<WARPS_M, WARPS_N, NSTAGES>, dim3(grid), dim3(WARPS_M * WARPS_N * 32), smem, stream, p);
+    RV_LAUNCH_ST = rv_launch(flash_paged_kernel<WARPS_M, WARPS_N, NSTAGES, DIST>, dim3(grid), dim3(WARPS_M * WARPS_N * 32), smem, stream, p);
     return rv_launch_status();
 }
 
@@ -1511,12 +1522,14 @@ RV_EXPORT long long rv_flash_scratch_floats(int n_tokens, int nh, int num_splits
 // the keys), for steps in which the selected sequences bring one token each.
 // scratch: float buffer of rv_flash_scratch_floats(...) elements when num_splits > 1.
 // `softcap` > 0: scaled scores pass softcap * tanh(s / softcap); `sinks` (float [nh]): exp(sink) joins each head's
-// softmax denominator; `gate` (float [n_tokens, nh]): multiplies each head's output.  Null / 0: absent.
+// softmax denominator; `gate` (float [n_tokens, nh]): multiplies each head's output; `dist` (float [nkv, dist_n, nh / nkv], in
+// units of log2): added to a score by the distance between query and key, after the cap.  Null / 0: absent.
 RV_EXPORT int rv_flash_attention_ex(const void* q, const void* cache, const int* block_tables, const int* cu_seqlens,
                                     const int* ctx_lens, void* out, float* scratch, int n_tokens, int num_seqs,
                                     int nh, int nkv, int hd, int page_size, int max_blocks, float scale, int window,
                                     int mode, int max_q_len, int num_splits, int q_filter, float softcap,
-                                    const float* sinks, const float* gate, cudaStream_t stream) {
+                                    const float* sinks, const float* gate, const float* dist, int dist_n, cudaStream_t stream) {
+    if (dist && dist_n <= 0) return RV_ERR_BAD_SIZE;
     if (hd != HEAD_DIM) return RV_ERR_UNSUPPORTED;
     if (n_tokens < 0 || num_seqs < 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || max_blocks <= 0 ||
         max_q_len <= 0 || num_splits < 1)
@@ -1541,10 +1554,15 @@ RV_EXPORT int rv_flash_attention_ex(const void* q, const void* cache, const int*
     p.cap_log2e = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     p.scale_over_cap = softcap > 0.f ? scale / softcap : 0.f;
     p.sinks = sinks; p.gate = gate;
+    p.dist = dist; p.dist_n = dist_n;
     const int G = nh / nkv;
     const int m_tile = mode == 1 ? 16 : 64;
     p.row_tiles = (max_q_len * G + m_tile - 1) / m_tile;
-    int st = mode == 1 ? launch_flash<1, 4, DECODE_STAGES>(p, num_seqs, stream) : launch_flash<4, 1, 2>(p, num_seqs, stream);
+    int st;
+    if (p.dist)
+        st = mode == 1 ? launch_flash<1, 4, DECODE_STAGES, true>(p, num_seqs, stream) : launch_flash<4, 1, 2, true>(p, num_seqs, stream);
+    else
+        st = mode == 1 ? launch_flash<1, 4, DECODE_STAGES>(p, num_seqs, stream) : launch_flash<4, 1, 2>(p, num_seqs, stream);
     if (st != RV_OK) return st;
     if (num_splits > 1) {
         RV_LAUNCH_ST = rv_launch(flash_combine_kernel, dim3((n_tokens * nh + COMBINE_ROWS - 1) / COMBINE_ROWS), dim3(128), 0, stream,
@@ -1560,7 +1578,7 @@ RV_EXPORT int rv_flash_attention(const void* q, const void* cache, const int* bl
                                  int mode, int max_q_len, int num_splits, int q_filter, cudaStream_t stream) {
     return rv_flash_attention_ex(q, cache, block_tables, cu_seqlens, ctx_lens, out, scratch, n_tokens, num_seqs, nh, nkv, hd,
                                  page_size, max_blocks, scale, window, mode, max_q_len, num_splits, q_filter, 0.f, nullptr,
-                                 nullptr, stream);
+                                 nullptr, nullptr, 0, stream);
 }
 
 // The TMA-fed decode kernel for the sequences of a step that bring one token (q_filter 1) or for
@@ -1572,8 +1590,10 @@ RV_EXPORT int rv_flash_decode_tma_ex(const void* q, const void* cache, long long
                                      const int* cu_seqlens, const int* ctx_lens, void* out, float* scratch, int n_tokens,
                                      int num_seqs, int nh, int nkv, int hd, int page_size, int max_blocks, float scale,
                                      int window, int max_q_len, int num_splits, int q_filter, int* status, int early,
-                                     float softcap, const float* sinks, const float* gate, cudaStream_t stream) {
+                                     float softcap, const float* sinks, const float* gate, const float* dist, int dist_n,
+                                     cudaStream_t stream) {
 #ifdef RV_HAVE_TMA_DECODE
+    if (dist && dist_n <= 0) return RV_ERR_BAD_SIZE;
     if (hd != HEAD_DIM) return RV_ERR_UNSUPPORTED;
     if (n_tokens < 0 || num_seqs < 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || max_blocks <= 0 ||
         max_q_len <= 0 || num_splits < 1 || num_pages <= 0)
@@ -1601,13 +1621,16 @@ RV_EXPORT int rv_flash_decode_tma_ex(const void* q, const void* cache, long long
     p.cap_log2e = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     p.scale_over_cap = softcap > 0.f ? scale / softcap : 0.f;
     p.sinks = sinks; p.gate = gate;
+    p.dist = dist; p.dist_n = dist_n;
     const int G = nh / nkv;
     p.row_tiles = (max_q_len * G + 15) / 16;
     const int smem = 2 * TMA_STAGES * TMA_TILE_BYTES + 1024;
     static RvPerDevice configured;
-    if (int e = rv_configure_smem(configured, flash_decode_tma_kernel<TMA_STAGES>, smem)) return e;
+    static RvPerDevice configured_dist;
+    auto kernel = dist ? flash_decode_tma_kernel<TMA_STAGES, true> : flash_decode_tma_kernel<TMA_STAGES, false>;
+    if (int e = rv_configure_smem(dist ? configured_dist : configured, kernel, smem)) return e;
     const dim3 grid(p.row_tiles * p.num_splits, p.nkv, num_seqs);
-    RV_LAUNCH_ST = rv_launch(flash_decode_tma_kernel<TMA_STAGES>, grid, dim3(TMA_THREADS), smem, stream, map_kv, p, status, early);
+    RV_LAUNCH_ST = rv_launch(kernel, grid, dim3(TMA_THREADS), smem, stream, map_kv, p, status, early);
     st = rv_launch_status();
     if (st != RV_OK) return st;
     if (num_splits > 1) {
@@ -1628,7 +1651,7 @@ RV_EXPORT int rv_flash_decode_tma(const void* q, const void* cache, long long nu
                                   cudaStream_t stream) {
     return rv_flash_decode_tma_ex(q, cache, num_pages, block_tables, cu_seqlens, ctx_lens, out, scratch, n_tokens, num_seqs, nh,
                                   nkv, hd, page_size, max_blocks, scale, window, max_q_len, num_splits, q_filter, status, early,
-                                  0.f, nullptr, nullptr, stream);
+                                  0.f, nullptr, nullptr, nullptr, 0, stream);
 }
 
 // The evenly cut decode kernel fed by TMA (head sizes 64 and 128, pages of at least 8 keys; else

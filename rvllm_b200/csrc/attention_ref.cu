@@ -11,7 +11,8 @@
 // Options for mixers that want them: `softcap` > 0 replaces a scaled score s by
 // softcap * tanh(s / softcap); `sinks` (one float per query head) adds exp(sink_h) to the softmax
 // denominator - a key without a value, neither scaled nor capped; `gate` (float [tokens, heads])
-// multiplies each head's output.
+// multiplies each head's output; `dist` (float [nkv, dist_n, nh / nkv]) is added to a (scaled, capped) score by the distance
+// between query and key, a distance beyond the last reading the last.
 //
 // Cache layer layout: [num_pages, planes, nkv, page_size, hd].  planes = 2: keys in plane 0, values in plane 1.
 // planes = 1: one row per token and kv head; the key is the whole row and the value its leading `vd` elements
@@ -26,7 +27,7 @@ __global__ void paged_attention_ref_kernel(const T* __restrict__ q, const T* __r
                                            T* __restrict__ out, int n_tokens, int nh, int nkv, int hd,
                                            int page_size, int max_blocks, float scale, int window,
                                            float softcap, const float* __restrict__ sinks, const float* __restrict__ gate,
-                                           int planes, int vd) {
+                                           int planes, int vd, const float* __restrict__ dist, int dist_n) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -57,6 +58,8 @@ __global__ void paged_attention_ref_kernel(const T* __restrict__ q, const T* __r
     }
     float m = -INFINITY, l = 0.f;
     const int* table = block_tables + (size_t)seq * max_blocks;
+    const int G = nh / nkv;
+    const float* bias = dist ? dist + (size_t)kvh * dist_n * G + (h - kvh * G) : nullptr;
     const size_t page_stride = (size_t)planes * nkv * page_size * hd;
     const size_t v_off = planes == 2 ? (size_t)nkv * page_size * hd : 0;
     for (int j = lo; j <= pos; ++j) {
@@ -71,6 +74,7 @@ __global__ void paged_attention_ref_kernel(const T* __restrict__ q, const T* __r
         }
         s = rv_warp_sum(s);
         if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+        if (bias) s += bias[(size_t)min(pos - j, dist_n - 1) * G];
         const float m_new = fmaxf(m, s);
         const float corr = expf(m - m_new);     // exp(-inf) = 0 at the first key
         const float p = expf(s - m_new);
@@ -103,17 +107,17 @@ template <int DPL>
 static int launch_ref(const void* q, const void* cache, const int* block_tables, const int* cu_seqlens, const int* ctx_lens,
                       const int* token_seq, void* out, int n_tokens, int nh, int nkv, int hd, int page_size, int max_blocks,
                       float scale, int window, float softcap, const float* sinks, const float* gate, int planes, int vd,
-                      int dtype, cudaStream_t stream) {
+                      int dtype, const float* dist, int dist_n, cudaStream_t stream) {
     const int warps = 4;
     const dim3 grid(n_tokens, (nh + warps - 1) / warps);
     if (dtype == RV_DTYPE_F32)
         RV_LAUNCH_ST = rv_launch(paged_attention_ref_kernel<float, DPL>, dim3(grid), dim3(warps * 32), 0, stream,
             (const float*)q, (const float*)cache, block_tables, cu_seqlens, ctx_lens, token_seq, (float*)out,
-            n_tokens, nh, nkv, hd, page_size, max_blocks, scale, window, softcap, sinks, gate, planes, vd);
+            n_tokens, nh, nkv, hd, page_size, max_blocks, scale, window, softcap, sinks, gate, planes, vd, dist, dist_n);
     else if (dtype == RV_DTYPE_BF16)
         RV_LAUNCH_ST = rv_launch(paged_attention_ref_kernel<__nv_bfloat16, DPL>, dim3(grid), dim3(warps * 32), 0, stream,
             (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, block_tables, cu_seqlens, ctx_lens, token_seq,
-            (__nv_bfloat16*)out, n_tokens, nh, nkv, hd, page_size, max_blocks, scale, window, softcap, sinks, gate, planes, vd);
+            (__nv_bfloat16*)out, n_tokens, nh, nkv, hd, page_size, max_blocks, scale, window, softcap, sinks, gate, planes, vd, dist, dist_n);
     else
         return RV_ERR_BAD_DTYPE;
     return rv_launch_status();
@@ -124,16 +128,18 @@ RV_EXPORT int rv_paged_attention_ref_ex(const void* q, const void* cache, const 
                                         const int* cu_seqlens, const int* ctx_lens, const int* token_seq,
                                         void* out, int n_tokens, int nh, int nkv, int hd, int page_size,
                                         int max_blocks, float scale, int window, float softcap, const float* sinks,
-                                        const float* gate, int planes, int vd, int dtype, cudaStream_t stream) {
+                                        const float* gate, int planes, int vd, int dtype, const float* dist, int dist_n,
+                                        cudaStream_t stream) {
+    if (dist && (dist_n <= 0 || nkv <= 0 || nh % nkv)) return RV_ERR_BAD_SIZE;
     if (n_tokens < 0 || nh <= 0 || nkv <= 0 || hd <= 0 || page_size <= 0 || max_blocks <= 0) return RV_ERR_BAD_SIZE;
     if ((planes != 1 && planes != 2) || vd <= 0 || vd > hd || (planes == 2 && vd != hd)) return RV_ERR_BAD_SIZE;
     if (hd > 32 * 32) return RV_ERR_UNSUPPORTED;
     if (n_tokens == 0) return RV_OK;
     if (hd <= 32 * 8)
         return launch_ref<8>(q, cache, block_tables, cu_seqlens, ctx_lens, token_seq, out, n_tokens, nh, nkv, hd, page_size,
-                             max_blocks, scale, window, softcap, sinks, gate, planes, vd, dtype, stream);
+                             max_blocks, scale, window, softcap, sinks, gate, planes, vd, dtype, dist, dist_n, stream);
     return launch_ref<32>(q, cache, block_tables, cu_seqlens, ctx_lens, token_seq, out, n_tokens, nh, nkv, hd, page_size,
-                          max_blocks, scale, window, softcap, sinks, gate, planes, vd, dtype, stream);
+                          max_blocks, scale, window, softcap, sinks, gate, planes, vd, dtype, dist, dist_n, stream);
 }
 
 RV_EXPORT int rv_paged_attention_ref(const void* q, const void* cache, const int* block_tables,
@@ -143,5 +149,5 @@ RV_EXPORT int rv_paged_attention_ref(const void* q, const void* cache, const int
                                      const float* gate, int dtype, cudaStream_t stream) {
     if (hd > 32 * 8) return RV_ERR_UNSUPPORTED;
     return rv_paged_attention_ref_ex(q, cache, block_tables, cu_seqlens, ctx_lens, token_seq, out, n_tokens, nh, nkv, hd,
-                                     page_size, max_blocks, scale, window, softcap, sinks, gate, 2, hd, dtype, stream);
+                                     page_size, max_blocks, scale, window, softcap, sinks, gate, 2, hd, dtype, nullptr, 0, stream);
 }

@@ -115,6 +115,10 @@ struct AttnParams {
     float scale_over_cap;          // scale / c
     const float* sinks;            // [nh] or null
     const float* gate;             // [n_tokens, nh] or null
+    // a bias per (distance, head) in units of log2, added after the cap: [nkv][dist_n][G], a distance beyond the last reads the
+    // last.  A row of the tile is (token, head in group), so the rows of a warp read neighbouring numbers.
+    const float* dist;             // or null
+    int dist_n;
 };
 
 __device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
@@ -175,6 +179,8 @@ __device__ __forceinline__ uint64_t umma_desc_mn(uint32_t smem_addr, uint32_t lb
     return d;
 }
 
+// DIST: the build with a bias per (distance, head)
+template <bool DIST>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                          const AttnParams p) {
@@ -426,6 +432,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         const int head = kvh * G + (in_range ? r - tok_i * G : 0);
         const int pos = in_range ? ctx - q_len + tok_i : -1;
         const int lo = (p.window > 0 && pos - p.window + 1 > 0) ? pos - p.window + 1 : 0;
+        const float* bias_row = DIST ? p.dist + (size_t)kvh * p.dist_n * G + (head - kvh * G) : nullptr;
+        const float bias_far = bias_row ? __ldg(bias_row + (size_t)(p.dist_n - 1) * G) : 0.f;
         const uint32_t t_lane = tmem_base + ((uint32_t)(warp * 32) << 16);
         float m_ref = -INFINITY, l_run = 0.f;
         bool ok = true;
@@ -450,7 +458,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             const int key0 = t * KV_TILE;
             // With a cap the scores become c log2(e) tanh(scale s / c) here (tanh as 1 - 2 / (e^2x + 1)), before the
             // masks, and the scale below is 1.
-            const float eff_scale = p.cap_log2e > 0.f ? 1.f : p.scale_log2e;
+            const float eff_scale = DIST || p.cap_log2e > 0.f ? 1.f : p.scale_log2e;
             if (p.cap_log2e > 0.f) {
                 const float k2 = p.scale_over_cap * 2.885390081777927f;
 #pragma unroll
@@ -458,6 +466,26 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                     const float ea = fast_exp2(__uint_as_float(s0[e]) * k2), eb = fast_exp2(__uint_as_float(s1[e]) * k2);
                     s0[e] = __float_as_uint(p.cap_log2e * (1.f - __fdividef(2.f, ea + 1.f)));
                     s1[e] = __float_as_uint(p.cap_log2e * (1.f - __fdividef(2.f, eb + 1.f)));
+                }
+            }
+            if constexpr (DIST) {
+                // the scaled (or capped) score plus its bias; a tile that lies wholly beyond the table's last distance for every
+                // row of the warp adds one number per row
+                const float sc = p.cap_log2e > 0.f ? 1.f : p.scale_log2e;
+                const int far_from = pos - (p.dist_n - 1);           // keys up to here read the last entry
+                if (__all_sync(0xffffffffu, key0 + KV_TILE - 1 <= far_from || pos < 0)) {
+#pragma unroll
+                    for (int e = 0; e < 32; ++e) {
+                        s0[e] = __float_as_uint(fmaf(__uint_as_float(s0[e]), sc, bias_far));
+                        s1[e] = __float_as_uint(fmaf(__uint_as_float(s1[e]), sc, bias_far));
+                    }
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 32; ++e) {
+                        const int da = min(max(pos - key0 - e, 0), p.dist_n - 1), db = min(max(pos - key0 - 32 - e, 0), p.dist_n - 1);
+                        s0[e] = __float_as_uint(fmaf(__uint_as_float(s0[e]), sc, __ldg(bias_row + da * G)));
+                        s1[e] = __float_as_uint(fmaf(__uint_as_float(s1[e]), sc, __ldg(bias_row + db * G)));
+                    }
                 }
             }
             // Scores stay raw in the registers; scale and reference maximum are applied in one FMA
@@ -626,12 +654,14 @@ RV_EXPORT int rv_attention_tcgen05_planes() { return KV_PLANES; }
 // the decode kernel).  Refuses (RV_ERR_UNSUPPORTED) what it is not built for: a head size other
 // than HEAD_DIM, a group of more than 128 heads, pages of fewer than 8 keys.
 // `softcap` > 0: scaled scores pass softcap * tanh(s / softcap); `sinks` (float [nh]): exp(sink) joins each head's softmax
-// denominator; `gate` (float [n_tokens, nh]): multiplies each head's output.  Null / 0: absent.
+// denominator; `gate` (float [n_tokens, nh]): multiplies each head's output; `dist` (float [nkv, dist_n, nh / nkv], in units of
+// log2): added to a score by the distance between query and key.  Null / 0: absent.
 RV_EXPORT int rv_attention_tcgen05_ex(const void* q, const void* cache, long long num_pages, const int* block_tables,
                                       const int* cu_seqlens, const int* ctx_lens, void* out, int n_tokens, int num_seqs,
                                       int nh, int nkv, int hd, int page_size, int max_blocks, float scale, int window,
                                       int max_q_len, int* status, float softcap, const float* sinks, const float* gate,
-                                      cudaStream_t stream) {
+                                      const float* dist, int dist_n, cudaStream_t stream) {
+    if (dist && dist_n <= 0) return RV_ERR_BAD_SIZE;
     if (hd != ROW_REAL) return RV_ERR_UNSUPPORTED;
     if (n_tokens < 0 || num_seqs < 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || max_blocks <= 0 || max_q_len <= 0)
         return RV_ERR_BAD_SIZE;
@@ -657,13 +687,16 @@ RV_EXPORT int rv_attention_tcgen05_ex(const void* q, const void* cache, long lon
     p.cap_log2e = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     p.scale_over_cap = softcap > 0.f ? scale / softcap : 0.f;
     p.sinks = sinks; p.gate = gate;
+    p.dist = dist; p.dist_n = dist_n;
     const int smem = Q_BYTES + NK * K_BYTES + NV * V_BYTES + 256;
     static RvPerDevice configured;
-    if (int e = rv_configure_smem(configured, attention_tcgen05_kernel, smem)) return e;
+    static RvPerDevice configured_dist;
+    auto kernel = dist ? attention_tcgen05_kernel<true> : attention_tcgen05_kernel<false>;
+    if (int e = rv_configure_smem(dist ? configured_dist : configured, kernel, smem)) return e;
     const int tile_tokens = ROWS / G;
     const dim3 grid(nkv, num_seqs, (max_q_len + tile_tokens - 1) / tile_tokens);
     if (grid.y > 65535 || grid.z > 65535) return RV_ERR_UNSUPPORTED;
-    RV_LAUNCH_ST = rv_launch(attention_tcgen05_kernel, grid, dim3(NUM_THREADS), smem, stream, map_q, map_kv, p);
+    RV_LAUNCH_ST = rv_launch(kernel, grid, dim3(NUM_THREADS), smem, stream, map_q, map_kv, p);
     return rv_launch_status();
 }
 
@@ -672,5 +705,5 @@ RV_EXPORT int rv_attention_tcgen05(const void* q, const void* cache, long long n
                                    int nh, int nkv, int hd, int page_size, int max_blocks, float scale, int window,
                                    int max_q_len, int* status, cudaStream_t stream) {
     return rv_attention_tcgen05_ex(q, cache, num_pages, block_tables, cu_seqlens, ctx_lens, out, n_tokens, num_seqs, nh, nkv, hd,
-                                   page_size, max_blocks, scale, window, max_q_len, status, 0.f, nullptr, nullptr, stream);
+                                   page_size, max_blocks, scale, window, max_q_len, status, 0.f, nullptr, nullptr, nullptr, 0, stream);
 }

@@ -7,6 +7,9 @@
 //                    [c | r] goes into the token's cache slot, the unrotated query parts into q_plain [T, nh, dq],
 //                    the rotated ones into columns R .. R + dr of q_row [T, nh, R + dr] (whose leading R columns
 //                    the absorbing product fills afterwards), sigmoid of the gate logits into a float array.
+//   latent_down      the same for queries that go through a low-rank row of their own: rows [cq': Rq | c': R | r: dr | gate logits];
+//                    cq = cq' / sqrt(mean(cq'^2) + eps) * wq is written as [T, Rq], c and r as above
+//   latent_queries   ... and the queries' part alone, from rows [q: nh x (dq + dr)]
 //   head_linear      out[t, h, :] = W[h] x[t, h, :] for W [nh, N, K]: the per-head products that move a head's key
 //                    up-projection onto its query and apply its value up-projection to the attended latent.
 //                    x and out are given with row and head strides (slices of wider rows).  bfloat16 operands with
@@ -24,21 +27,72 @@ __device__ __forceinline__ void lt_store(void* p, int dtype, size_t i, float v) 
     else ((__nv_bfloat16*)p)[i] = __float2bfloat16_rn(v);
 }
 
-// One block per token.
+// queries of one token: per head dq plain elements, then dr rotated ones (dr - half items: a pair or a single element)
+__device__ __forceinline__ void lt_queries(const void* __restrict__ proj, int in_dtype, size_t row, int t, const float* cs, const float* sn,
+                                           int half, int halves, void* __restrict__ q_plain, void* __restrict__ q_row, int out_dtype,
+                                           int nh, int dq, int dr, int R) {
+    const int per_head = dq + dr - half, D = R + dr;
+    for (int item = threadIdx.x; item < nh * per_head; item += blockDim.x) {
+        const int h = item / per_head, i = item - h * per_head;
+        const size_t src = row + (size_t)h * (dq + dr);
+        if (i < dq) {
+            lt_store(q_plain, out_dtype, ((size_t)t * nh + h) * dq + i, lt_load(proj, in_dtype, src + i));
+            continue;
+        }
+        const int k = i - dq;
+        const size_t dst = ((size_t)t * nh + h) * D + R;
+        if (k < half) {
+            const int ia = halves ? k : 2 * k, ib = halves ? k + half : 2 * k + 1;
+            const float a = lt_load(proj, in_dtype, src + dq + ia), b = lt_load(proj, in_dtype, src + dq + ib);
+            const float c = cs[k], s = sn[k];
+            lt_store(q_row, out_dtype, dst + ia, a * c - b * s);
+            lt_store(q_row, out_dtype, dst + ib, b * c + a * s);
+        } else {
+            const int j = k + half;
+            lt_store(q_row, out_dtype, dst + j, lt_load(proj, in_dtype, src + dq + j));
+        }
+    }
+}
+
+__global__ void __launch_bounds__(256)
+latent_queries_kernel(const void* __restrict__ q, int in_dtype, const int* __restrict__ positions, const float* __restrict__ cos_t,
+                      const float* __restrict__ sin_t, int rot, int table_rows, int halves, void* __restrict__ q_plain,
+                      void* __restrict__ q_row, int out_dtype, int nh, int dq, int dr, int R) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    const int t = blockIdx.x, half = rot >> 1;
+    int pos = positions[t];
+    if (pos < 0) pos = 0;
+    if (pos >= table_rows) pos = table_rows - 1;      // the host refuses such positions; never read outside
+    const float* cs = cos_t ? cos_t + (size_t)pos * half : nullptr;
+    const float* sn = sin_t ? sin_t + (size_t)pos * half : nullptr;
+    lt_queries(q, in_dtype, (size_t)t * nh * (dq + dr), t, cs, sn, half, halves, q_plain, q_row, out_dtype, nh, dq, dr, R);
+}
+
+// One block per token.  Rq > 0: the row starts with a low-rank row of the queries instead of the queries (low_out [T, Rq]).
 __global__ void __launch_bounds__(256)
 latent_prepare_kernel(const void* __restrict__ proj, int in_dtype, int row_stride, const void* __restrict__ c_gamma, int gamma_dtype,
                       const int* __restrict__ positions, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                       int rot, int table_rows, const int* __restrict__ slot_mapping, void* __restrict__ cache,
                       void* __restrict__ q_plain, void* __restrict__ q_row, int out_dtype, float* __restrict__ gate_out,
-                      int nh, int dq, int dr, int R, float eps, int write_kv, int halves) {
+                      int nh, int dq, int dr, int R, float eps, int write_kv, int halves, int Rq, const void* __restrict__ q_gamma,
+                      int q_gamma_dtype, void* __restrict__ low_out) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     __shared__ float scratch[33];
     const int t = blockIdx.x;
     const size_t row = (size_t)t * row_stride;
-    const int qw = nh * (dq + dr), D = R + dr;
+    const int qw = Rq > 0 ? Rq : nh * (dq + dr), D = R + dr;
     const size_t c0 = row + qw;
     float ss = 0.f;
+    if (Rq > 0) {
+        for (int i = threadIdx.x; i < Rq; i += blockDim.x) { const float v = lt_load(proj, in_dtype, row + i); ss = fmaf(v, v, ss); }
+        ss = rv_block_sum(ss, scratch);
+        const float rq = 1.0f / sqrtf(ss / (float)Rq + eps);
+        for (int i = threadIdx.x; i < Rq; i += blockDim.x)
+            lt_store(low_out, out_dtype, (size_t)t * Rq + i, lt_load(proj, in_dtype, row + i) * rq * rv_load_param(q_gamma, q_gamma_dtype, i));
+        ss = 0.f;
+    }
     for (int i = threadIdx.x; i < R; i += blockDim.x) { const float v = lt_load(proj, in_dtype, c0 + i); ss = fmaf(v, v, ss); }
     ss = rv_block_sum(ss, scratch);
     const float rc = 1.0f / sqrtf(ss / (float)R + eps);
@@ -67,28 +121,7 @@ latent_prepare_kernel(const void* __restrict__ proj, int in_dtype, int row_strid
             }
         }
     }
-    // queries: per head dq plain elements, then dr rotated ones (dr - half items: a pair or a single element)
-    const int per_head = dq + dr - half;
-    for (int item = threadIdx.x; item < nh * per_head; item += blockDim.x) {
-        const int h = item / per_head, i = item - h * per_head;
-        const size_t src = row + (size_t)h * (dq + dr);
-        if (i < dq) {
-            lt_store(q_plain, out_dtype, ((size_t)t * nh + h) * dq + i, lt_load(proj, in_dtype, src + i));
-            continue;
-        }
-        const int k = i - dq;
-        const size_t dst = ((size_t)t * nh + h) * D + R;
-        if (k < half) {
-            const int ia = halves ? k : 2 * k, ib = halves ? k + half : 2 * k + 1;
-            const float a = lt_load(proj, in_dtype, src + dq + ia), b = lt_load(proj, in_dtype, src + dq + ib);
-            const float c = cs[k], s = sn[k];
-            lt_store(q_row, out_dtype, dst + ia, a * c - b * s);
-            lt_store(q_row, out_dtype, dst + ib, b * c + a * s);
-        } else {
-            const int j = k + half;
-            lt_store(q_row, out_dtype, dst + j, lt_load(proj, in_dtype, src + dq + j));
-        }
-    }
+    if (q_plain) lt_queries(proj, in_dtype, row, t, cs, sn, half, halves, q_plain, q_row, out_dtype, nh, dq, dr, R);
     if (gate_out)
         for (int h = threadIdx.x; h < nh; h += blockDim.x) {
             const float g = lt_load(proj, in_dtype, row + qw + D + h);
@@ -108,7 +141,37 @@ RV_EXPORT int rv_latent_prepare(const void* proj, int in_dtype, int row_stride, 
     if (!cos_t || !sin_t) rot = 0;
     RV_LAUNCH_ST = rv_launch(latent_prepare_kernel, dim3(n_tokens), dim3(256), 0, stream, proj, in_dtype, row_stride, c_gamma,
                              gamma_dtype, positions, cos_t, sin_t, rot, table_rows, slot_mapping, cache, q_plain, q_row, out_dtype,
-                             gate_out, nh, dq, dr, R, eps, write_kv, halves);
+                             gate_out, nh, dq, dr, R, eps, write_kv, halves, 0, (const void*)nullptr, 0, (void*)nullptr);
+    return rv_launch_status();
+}
+
+// gate_out null: no gate logits in the row (nh is then of no use).
+RV_EXPORT int rv_latent_down(const void* proj, int in_dtype, int row_stride, const void* q_gamma, int q_gamma_dtype, const void* c_gamma,
+                             int gamma_dtype, const int* positions, const float* cos_t, const float* sin_t, int rot, int table_rows,
+                             const int* slot_mapping, void* cache, void* low_out, int out_dtype, float* gate_out, int n_tokens, int nh,
+                             int Rq, int dr, int R, float eps, int write_kv, int halves, cudaStream_t stream) {
+    if (n_tokens < 0 || nh < 0 || Rq <= 0 || dr < 0 || R <= 0 || table_rows <= 0 || !low_out || !q_gamma) return RV_ERR_BAD_SIZE;
+    if (rot < 0 || rot > dr || (rot & 1)) return RV_ERR_BAD_SIZE;
+    if (row_stride < Rq + R + dr + (gate_out ? nh : 0)) return RV_ERR_BAD_SIZE;
+    if ((in_dtype | gamma_dtype | q_gamma_dtype | out_dtype) & ~1) return RV_ERR_BAD_DTYPE;
+    if (n_tokens == 0) return RV_OK;
+    if (!cos_t || !sin_t) rot = 0;
+    RV_LAUNCH_ST = rv_launch(latent_prepare_kernel, dim3(n_tokens), dim3(256), 0, stream, proj, in_dtype, row_stride, c_gamma,
+                             gamma_dtype, positions, cos_t, sin_t, rot, table_rows, slot_mapping, cache, (void*)nullptr, (void*)nullptr,
+                             out_dtype, gate_out, nh, 0, dr, R, eps, write_kv, halves, Rq, q_gamma, q_gamma_dtype, low_out);
+    return rv_launch_status();
+}
+
+RV_EXPORT int rv_latent_queries(const void* q, int in_dtype, const int* positions, const float* cos_t, const float* sin_t, int rot,
+                                int table_rows, void* q_plain, void* q_row, int out_dtype, int n_tokens, int nh, int dq, int dr, int R,
+                                int halves, cudaStream_t stream) {
+    if (n_tokens < 0 || nh <= 0 || dq <= 0 || dr < 0 || R <= 0 || table_rows <= 0) return RV_ERR_BAD_SIZE;
+    if (rot < 0 || rot > dr || (rot & 1)) return RV_ERR_BAD_SIZE;
+    if ((in_dtype | out_dtype) & ~1) return RV_ERR_BAD_DTYPE;
+    if (n_tokens == 0) return RV_OK;
+    if (!cos_t || !sin_t) { cos_t = sin_t = nullptr; rot = 0; }
+    RV_LAUNCH_ST = rv_launch(latent_queries_kernel, dim3(n_tokens), dim3(256), 0, stream, q, in_dtype, positions, cos_t, sin_t, rot,
+                             table_rows, halves, q_plain, q_row, out_dtype, nh, dq, dr, R);
     return rv_launch_status();
 }
 

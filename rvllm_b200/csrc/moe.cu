@@ -4,12 +4,14 @@
 //
 // Layout: gate_up [experts, 2 ff, width] (an expert's gate rows, then its up rows; plain experts: up [experts, ff, width]),
 // down [experts, width, ff], chosen [tokens, top] int32 expert numbers (numbers outside 0 .. experts-1 contribute
-// nothing), weights float [tokens, top] or null.
+// nothing - or, with `identity`, numbers from `experts` on contribute the token's own vector x_t), weights float
+// [tokens, top] or null.
 //
 //   moe_route_top act on a router's float32 logits: s = sigmoid(z); the choice is made among s + correction, within the best
 //                 `keep` of `groups` equal groups of neighbouring experts (a group counts by the sum of its two largest
-//                 corrected scores); chosen [tokens, top], weights = the chosen s over their sum (+ eps).  With `softmax`
-//                 the choice is made among z + correction itself and the weights are the softmax over the chosen ones
+//                 corrected scores - or, with `group_max`, by the largest); chosen [tokens, top], weights = the chosen s over
+//                 their sum (+ eps).  Mode 1: the choice is made among z + correction itself and the weights are the softmax
+//                 over the chosen ones.  Mode 2: as mode 0 with s = softmax(z) over all experts
 //   moe_gate_up   act[t * top + k, f] = silu(gate_e[f] . x_t) * (up_e[f] . x_t)  or  relu(up_e[f] . x_t)^2,  e = chosen[t, k]
 //   moe_down      out[t, n] = (add_scale[t] add[t, n]) + weight * sum_k weights[t, k] down_e(k)[n] . act[t * top + k]
 //
@@ -134,7 +136,7 @@ template <typename T, typename TO>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
 moe_down_kernel(const T* __restrict__ act, const int* __restrict__ chosen, const T* __restrict__ down, const float* add,
                 TO* out, int top, int experts, int ff, int width, float weight, const float* __restrict__ weights,
-                const float* __restrict__ add_scale) {
+                const float* __restrict__ add_scale, const T* __restrict__ identity_x) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     extern __shared__ float as[];                 // [top][ff]
@@ -148,6 +150,13 @@ moe_down_kernel(const T* __restrict__ act, const int* __restrict__ chosen, const
     for (int j = 0; j < MOE_PER_WARP; ++j) sum[j] = 0.f;
     for (int k = 0; k < top; ++k) {                       // the slots in their order: one sum per element, whatever the batch
         const int e = chosen[t * top + k];
+        if (e >= experts && identity_x) {
+            const float wk = weights ? weights[t * top + k] : 1.f;
+#pragma unroll
+            for (int j = 0; j < MOE_PER_WARP; ++j)
+                sum[j] = fmaf(wk, rv_to_float(identity_x[(size_t)t * width + min(width - 1, n0 + warp + j * MOE_WARPS)]), sum[j]);
+            continue;
+        }
         if (e < 0 || e >= experts) continue;
         const T* rows[MOE_PER_WARP];
 #pragma unroll
@@ -174,7 +183,7 @@ static RvPerDevice g_once[8];
 template <typename T>
 static int moe_launch(const void* x, const int* chosen, const float* weights, const void* gate_up, const void* down, void* act,
                       const float* add, const float* add_scale, void* out, int out_f32, int tokens, int top, int experts, int ff,
-                      int width, float weight, int gated, int slot, cudaStream_t stream) {
+                      int width, float weight, int gated, int identity, int slot, cudaStream_t stream) {
     const int smem_a = width * 4, smem_b = top * ff * 4;
     if (smem_a > 200 * 1024 || smem_b > 200 * 1024) return RV_ERR_UNSUPPORTED;
     int st;
@@ -197,12 +206,14 @@ static int moe_launch(const void* x, const int* chosen, const float* weights, co
         st = rv_configure_smem(g_once[slot + 1], moe_down_kernel<T, float>, 200 * 1024);
         if (st != RV_OK) return st;
         RV_LAUNCH_ST = rv_launch(moe_down_kernel<T, float>, dim3(grid), dim3(MOE_WARPS * 32), (size_t)smem_b, stream, (const T*)act,
-                                 chosen, (const T*)down, add, (float*)out, top, experts, ff, width, weight, weights, add_scale);
+                                 chosen, (const T*)down, add, (float*)out, top, experts, ff, width, weight, weights, add_scale,
+                                 identity ? (const T*)x : (const T*)nullptr);
     } else {
         st = rv_configure_smem(g_once[slot + 2], moe_down_kernel<T, T>, 200 * 1024);
         if (st != RV_OK) return st;
         RV_LAUNCH_ST = rv_launch(moe_down_kernel<T, T>, dim3(grid), dim3(MOE_WARPS * 32), (size_t)smem_b, stream, (const T*)act,
-                                 chosen, (const T*)down, add, (T*)out, top, experts, ff, width, weight, weights, add_scale);
+                                 chosen, (const T*)down, add, (T*)out, top, experts, ff, width, weight, weights, add_scale,
+                                 identity ? (const T*)x : (const T*)nullptr);
     }
     return rv_launch_status();
 }
@@ -213,22 +224,23 @@ static int moe_launch(const void* x, const int* chosen, const float* weights, co
 // first matrix is [gate | up] with SiLU, 0 it is the up matrix with a squared relu.  Two launches.
 RV_EXPORT int rv_moe_experts_ex(const void* x, const int* chosen, const float* weights, const void* gate_up, const void* down, void* act,
                                 const float* add, const float* add_scale, void* out, int out_f32, int tokens, int top, int experts,
-                                int ff, int width, float weight, int gated, int dtype, cudaStream_t stream) {
+                                int ff, int width, float weight, int gated, int identity, int dtype, cudaStream_t stream) {
     if (tokens < 0 || top <= 0 || experts <= 0 || ff <= 0 || width <= 0) return RV_ERR_BAD_SIZE;
     if ((long long)tokens * top > 0x7fffffffLL || ff > 65535 * MOE_FEATURES || width > 65535 * MOE_FEATURES) return RV_ERR_BAD_SIZE;
     if (tokens == 0) return RV_OK;
     if (dtype == RV_DTYPE_F32)
-        return moe_launch<float>(x, chosen, weights, gate_up, down, act, add, add_scale, out, 1, tokens, top, experts, ff, width, weight, gated, 0, stream);
+        return moe_launch<float>(x, chosen, weights, gate_up, down, act, add, add_scale, out, 1, tokens, top, experts, ff, width, weight, gated, identity, 0,
+                                 stream);
     if (dtype == RV_DTYPE_BF16)
         return moe_launch<__nv_bfloat16>(x, chosen, weights, gate_up, down, act, add, add_scale, out, out_f32, tokens, top, experts, ff, width,
-                                         weight, gated, 4, stream);
+                                         weight, gated, identity, 4, stream);
     return RV_ERR_BAD_DTYPE;
 }
 
 RV_EXPORT int rv_moe_experts(const void* x, const int* chosen, const void* gate_up, const void* down, void* act, const float* add,
                              void* out, int out_f32, int tokens, int top, int experts, int ff, int width, float weight,
                              int dtype, cudaStream_t stream) {
-    return rv_moe_experts_ex(x, chosen, nullptr, gate_up, down, act, add, nullptr, out, out_f32, tokens, top, experts, ff, width, weight, 1,
+    return rv_moe_experts_ex(x, chosen, nullptr, gate_up, down, act, add, nullptr, out, out_f32, tokens, top, experts, ff, width, weight, 1, 0,
                              dtype, stream);
 }
 
@@ -310,7 +322,8 @@ __global__ void moe_gather_kernel(const uint4* __restrict__ x, const int* __rest
 template <typename TO>
 __global__ void moe_combine_kernel(const float* __restrict__ ys, const int* __restrict__ row_of, const float* add, TO* out,
                                    int top, int width, float weight, size_t total, const float* __restrict__ weights,
-                                   const float* __restrict__ add_scale) {
+                                   const float* __restrict__ add_scale, const __nv_bfloat16* __restrict__ identity_x,
+                                   const int* __restrict__ chosen, int experts) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
@@ -320,6 +333,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ ys, const int* __re
         for (int k = 0; k < top; ++k) {
             const int row = row_of[t * top + k];
             if (row >= 0) s = fmaf(weights ? weights[t * top + k] : 1.f, ys[(size_t)row * width + n], s);
+            else if (identity_x && chosen[t * top + k] >= experts)
+                s = fmaf(weights ? weights[t * top + k] : 1.f, __bfloat162float(identity_x[i]), s);
         }
         float v = s * weight;
         if (add) v += add_scale ? add_scale[t] * add[i] : add[i];
@@ -350,16 +365,19 @@ RV_EXPORT int rv_moe_gather(const void* x, const int* src_of, void* xs, int rows
 }
 
 RV_EXPORT int rv_moe_combine(const float* ys, const int* row_of, const float* add, void* out, int out_f32, int tokens, int top,
-                             int width, float weight, const float* weights, const float* add_scale, cudaStream_t stream) {
+                             int width, float weight, const float* weights, const float* add_scale, const void* identity_x,
+                             const int* chosen, int experts, cudaStream_t stream) {
+    if (identity_x && (!chosen || experts <= 0)) return RV_ERR_BAD_SIZE;
     if (tokens < 0 || top <= 0 || width <= 0) return RV_ERR_BAD_SIZE;
     if (tokens == 0) return RV_OK;
     const size_t total = (size_t)tokens * width;
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     if (out_f32)
-        RV_LAUNCH_ST = rv_launch(moe_combine_kernel<float>, dim3(blocks), dim3(256), 0, stream, ys, row_of, add, (float*)out, top, width, weight, total, weights, add_scale);
+        RV_LAUNCH_ST = rv_launch(moe_combine_kernel<float>, dim3(blocks), dim3(256), 0, stream, ys, row_of, add, (float*)out, top, width, weight, total, weights, add_scale,
+                                 (const __nv_bfloat16*)identity_x, chosen, experts);
     else
         RV_LAUNCH_ST = rv_launch(moe_combine_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, ys, row_of, add, (__nv_bfloat16*)out, top,
-                                 width, weight, total, weights, add_scale);
+                                 width, weight, total, weights, add_scale, (const __nv_bfloat16*)identity_x, chosen, experts);
     return rv_launch_status();
 }
 
@@ -384,7 +402,7 @@ __device__ __forceinline__ void mr_argmax(const float* v, int n, int lane, float
 __global__ void __launch_bounds__(MR_WARPS * 32)
 moe_route_top_kernel(const float* __restrict__ logits, int stride, const float* __restrict__ correction, int* __restrict__ chosen,
                      float* __restrict__ weights, float* __restrict__ gate_out, int tokens, int experts, int top, int groups, int keep,
-                     float weight_eps, int softmax) {
+                     float weight_eps, int mode, int group_max) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     extern __shared__ float mr_smem[];
@@ -395,28 +413,39 @@ moe_route_top_kernel(const float* __restrict__ logits, int stride, const float* 
     float* c = s + experts;
     float* gs = c + experts;
     const float* z = logits + (size_t)t * stride;
-    for (int e = lane; e < experts; e += 32) {
-        const float v = softmax ? z[e] + correction[e] : 1.0f / (1.0f + expf(-z[e]));
-        s[e] = v;
-        c[e] = softmax ? v : v + correction[e];
+    const bool softmax = mode == 1;
+    if (mode == 2) {                                        // a softmax over all experts; every lane keeps to its own entries
+        float most = -INFINITY, total = 0.f;
+        for (int e = lane; e < experts; e += 32) most = fmaxf(most, z[e]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) most = fmaxf(most, __shfl_xor_sync(0xffffffffu, most, o));
+        for (int e = lane; e < experts; e += 32) { s[e] = expf(z[e] - most); total += s[e]; }
+        total = rv_warp_sum(total);
+        for (int e = lane; e < experts; e += 32) { s[e] = s[e] / total; c[e] = s[e] + correction[e]; }
+    } else {
+        for (int e = lane; e < experts; e += 32) {
+            const float v = softmax ? z[e] + correction[e] : 1.0f / (1.0f + expf(-z[e]));
+            s[e] = v;
+            c[e] = softmax ? v : v + correction[e];
+        }
     }
     if (gate_out && lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-z[experts]));
     __syncwarp();
     if (keep < groups) {
         const int per = experts / groups;
-        for (int g = lane; g < groups; g += 32) {           // a group counts by its two largest corrected scores
+        for (int g = lane; g < groups; g += 32) {           // a group counts by its two largest corrected scores, or the largest
             float a = -INFINITY, b = -INFINITY;
             for (int i = 0; i < per; ++i) {
                 const float v = c[g * per + i];
                 if (v > a) { b = a; a = v; } else if (v > b) b = v;
             }
-            gs[g] = per > 1 ? a + b : a;
+            gs[g] = per > 1 && !group_max ? a + b : a;
         }
         __syncwarp();
         for (int k = 0; k < keep; ++k) {                    // the kept groups are marked +inf, then the others are closed
             float best; int at;
             mr_argmax(gs, groups, lane, best, at);
-            if (lane == 0) gs[at] = -INFINITY;
+            if (lane == 0 && at < groups) gs[at] = -INFINITY;
             __syncwarp();
         }
         for (int e = lane; e < experts; e += 32)
@@ -447,7 +476,8 @@ moe_route_top_kernel(const float* __restrict__ logits, int stride, const float* 
 
 // logits float [tokens, stride]: the experts' logits and, with gate_out, one more column whose sigmoid goes to gate_out.
 RV_EXPORT int rv_moe_route_top(const float* logits, int stride, const float* correction, int* chosen, float* weights, float* gate_out,
-                               int tokens, int experts, int top, int groups, int keep, float weight_eps, int softmax, cudaStream_t stream) {
+                               int tokens, int experts, int top, int groups, int keep, float weight_eps, int mode, int group_max, cudaStream_t stream) {
+    if (mode < 0 || mode > 2) return RV_ERR_UNSUPPORTED;
     if (tokens < 0 || experts <= 0 || top <= 0 || top > experts || groups <= 0 || experts % groups || keep <= 0 || keep > groups)
         return RV_ERR_BAD_SIZE;
     if (stride < experts + (gate_out ? 1 : 0) || top > (experts / groups) * keep) return RV_ERR_BAD_SIZE;
@@ -455,6 +485,6 @@ RV_EXPORT int rv_moe_route_top(const float* logits, int stride, const float* cor
     if (tokens == 0) return RV_OK;
     const size_t smem = (size_t)MR_WARPS * (2 * experts + groups) * sizeof(float);
     RV_LAUNCH_ST = rv_launch(moe_route_top_kernel, dim3((tokens + MR_WARPS - 1) / MR_WARPS), dim3(MR_WARPS * 32), smem, stream, logits,
-                             stride, correction, chosen, weights, gate_out, tokens, experts, top, groups, keep, weight_eps, softmax);
+                             stride, correction, chosen, weights, gate_out, tokens, experts, top, groups, keep, weight_eps, mode, group_max);
     return rv_launch_status();
 }

@@ -11,8 +11,14 @@
 //                     its d elements at m d, a key row all maps side by side, so that (query row of map m) . (key row) is
 //                     map m's score; everything else of a row is written as zeros.  sigmoid of the gate logits goes to a
 //                     float array.  A token with slot -1 writes no key and no value.
+//                     Options: weighted norms instead of the unit norm, x / sqrt(mean(x^2) + eps) * gamma IN FRONT of the
+//                     rotation (one gamma of d elements for the queries, one for the keys); a factor
+//                     1 + coef ln(floor((p + 1) / every) + 1) on the query of position p; the value as projected kept in a
+//                     float array, or (1 - lambda) of the value plus lambda of such an array's row
 //   turn_back         rows of attention results [T, nh, P]: the leading vd elements of every head turned by MINUS the token's
 //                     angle, written as [T, nh, vd]
+//   gate_elements     rows of attention results [T, nh, P]: the leading vd elements of every head times the sigmoid of a float
+//                     logit of their own, written as [T, nh, vd]
 //   map_difference    rows [T, nh, 2, P] of two maps' results: o = a1 - lambda a2 over the leading vd elements, then
 //                     o / sqrt(mean(o^2) + eps) * factor, written as [T, nh, vd]
 //
@@ -34,6 +40,9 @@ struct QkPrepareArgs {
     const float *vcos_t, *vsin_t; int v_table_rows;            // value tables [rows, vd / 2] or null
     const int* slot_mapping; void *cache, *q_out; int out_dtype; float* gate_out;
     int nh, nkv, d, vd, P, maps, page_size; float eps; int unit, write_kv;
+    const float *q_gamma, *k_gamma;                             // [d] each: weighted norms in front of the rotation, or null
+    float temp_coef; int temp_every;                            // temp_every 0: no temperature
+    float* keep_v; const float* mix_v; float lambda;            // [T, nkv x vd] each, or null
 };
 
 // Element e of a vector of which the leading `rot` elements turn; `cs` and `sn` are the token's rows of the tables.
@@ -78,12 +87,28 @@ qk_prepare_kernel(const QkPrepareArgs a) {
     for (int item = warp; item < items; item += QP_WARPS) {
         const int kind = item < nq ? 0 : (item < nq + nk ? 1 : 2);            // q, k, v
         const int index = kind == 0 ? item : (kind == 1 ? item - nq : item - nq - nk);
-        if (kind != 0 && slot < 0) continue;                                  // (the same for the whole warp)
+        if (kind != 0 && slot < 0 && !(kind == 2 && a.keep_v)) continue;      // (the same for the whole warp)
         const int n = kind == 2 ? a.vd : a.d;
         const int head = kind == 2 ? index : index / a.maps, map = kind == 2 ? 0 : index - head * a.maps;
         const size_t col = kind == 0 ? (size_t)index * a.d
                                      : (kind == 1 ? (size_t)(nq + index) * a.d : (size_t)(nq + nk) * a.d + (size_t)index * a.vd);
-        for (int i = lane; i < n; i += 32) mine[i] = a.proj[row + col + i] + (a.bias ? a.bias[col + i] : 0.f);
+        const float* gamma = kind == 0 ? a.q_gamma : (kind == 1 ? a.k_gamma : nullptr);
+        float before = 0.f;
+        for (int i = lane; i < n; i += 32) {
+            float v = a.proj[row + col + i] + (a.bias ? a.bias[col + i] : 0.f);
+            if (kind == 2) {
+                const size_t at = ((size_t)t * a.nkv + index) * a.vd + i;
+                if (a.keep_v) a.keep_v[at] = v;
+                if (a.mix_v) v = (1.0f - a.lambda) * v + a.lambda * a.mix_v[at];
+            }
+            mine[i] = v;
+            before = fmaf(v, v, before);
+        }
+        if (kind != 0 && slot < 0) continue;
+        if (gamma) {                                                          // a lane scales what it has stored itself
+            const float g = 1.0f / sqrtf(rv_warp_sum(before) / (float)n + a.eps);
+            for (int i = lane; i < n; i += 32) mine[i] = mine[i] * g * gamma[i];
+        }
         __syncwarp();
         const float* c = kind == 2 ? vcs : cs;
         const float* s = kind == 2 ? vsn : sn;
@@ -103,6 +128,7 @@ qk_prepare_kernel(const QkPrepareArgs a) {
             ss = rv_warp_sum(ss);
             r = 1.0f / sqrtf(ss / (float)n + a.eps);
         }
+        if (kind == 0 && a.temp_every > 0) r *= 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1));
         void* dst_base;
         size_t dst;
         if (kind == 0) {
@@ -129,11 +155,15 @@ qk_prepare_kernel(const QkPrepareArgs a) {
     }
 }
 
-RV_EXPORT int rv_qk_prepare(const float* proj, int row_stride, const float* bias, const int* positions, const float* cos_t,
-                            const float* sin_t, int rot, int table_rows, int halves, const float* vcos_t, const float* vsin_t,
-                            int v_table_rows, const int* slot_mapping, void* cache, void* q_out, int out_dtype, float* gate_out,
-                            int n_tokens, int nh, int nkv, int d, int vd, int P, int maps, int page_size, float eps, int unit,
-                            int write_kv, cudaStream_t stream) {
+// q_gamma and k_gamma go together and exclude `unit`; keep_v and mix_v are float [n_tokens, nkv * vd].
+RV_EXPORT int rv_qk_prepare_ex(const float* proj, int row_stride, const float* bias, const int* positions, const float* cos_t,
+                               const float* sin_t, int rot, int table_rows, int halves, const float* vcos_t, const float* vsin_t,
+                               int v_table_rows, const int* slot_mapping, void* cache, void* q_out, int out_dtype, float* gate_out,
+                               int n_tokens, int nh, int nkv, int d, int vd, int P, int maps, int page_size, float eps, int unit,
+                               int write_kv, const float* q_gamma, const float* k_gamma, float temp_coef, int temp_every,
+                               float* keep_v, const float* mix_v, float lambda, cudaStream_t stream) {
+    if ((q_gamma == nullptr) != (k_gamma == nullptr) || (q_gamma && unit) || temp_every < 0) return RV_ERR_BAD_SIZE;
+    if ((keep_v || mix_v) && !write_kv) return RV_ERR_BAD_SIZE;
     if (n_tokens < 0 || nh <= 0 || nkv <= 0 || d <= 0 || vd <= 0 || P < vd || page_size <= 0 || table_rows <= 0 || v_table_rows <= 0)
         return RV_ERR_BAD_SIZE;
     if (maps != 1 && maps != 2) return RV_ERR_BAD_SIZE;
@@ -147,11 +177,22 @@ RV_EXPORT int rv_qk_prepare(const float* proj, int row_stride, const float* bias
     if (n_tokens == 0) return RV_OK;
     if (!cos_t || !sin_t) { cos_t = sin_t = nullptr; rot = 0; }
     const QkPrepareArgs a = {proj, row_stride, bias, positions, cos_t, sin_t, rot, table_rows, halves, vcos_t, vsin_t, v_table_rows,
-                             slot_mapping, cache, q_out, out_dtype, gate_out, nh, nkv, d, vd, P, maps, page_size, eps, unit, write_kv};
+                             slot_mapping, cache, q_out, out_dtype, gate_out, nh, nkv, d, vd, P, maps, page_size, eps, unit, write_kv,
+                             q_gamma, k_gamma, temp_coef, temp_every, keep_v, mix_v, lambda};
     auto kernel = P <= 32 ? qk_prepare_kernel<1> : (P <= 64 ? qk_prepare_kernel<2> : (P <= 128 ? qk_prepare_kernel<4>
                 : (P <= 256 ? qk_prepare_kernel<8> : qk_prepare_kernel<32>)));
     RV_LAUNCH_ST = rv_launch(kernel, dim3(n_tokens), dim3(QP_WARPS * 32), 0, stream, a);
     return rv_launch_status();
+}
+
+RV_EXPORT int rv_qk_prepare(const float* proj, int row_stride, const float* bias, const int* positions, const float* cos_t,
+                            const float* sin_t, int rot, int table_rows, int halves, const float* vcos_t, const float* vsin_t,
+                            int v_table_rows, const int* slot_mapping, void* cache, void* q_out, int out_dtype, float* gate_out,
+                            int n_tokens, int nh, int nkv, int d, int vd, int P, int maps, int page_size, float eps, int unit,
+                            int write_kv, cudaStream_t stream) {
+    return rv_qk_prepare_ex(proj, row_stride, bias, positions, cos_t, sin_t, rot, table_rows, halves, vcos_t, vsin_t, v_table_rows,
+                            slot_mapping, cache, q_out, out_dtype, gate_out, n_tokens, nh, nkv, d, vd, P, maps, page_size, eps, unit,
+                            write_kv, nullptr, nullptr, 0.f, 0, nullptr, nullptr, 0.f, stream);
 }
 
 // ------------------------------------------------------------------ after the attention kernels
@@ -239,6 +280,43 @@ RV_EXPORT int rv_turn_back(const void* o, const int* positions, const float* cos
     else
         RV_LAUNCH_ST = rv_launch(turn_back_kernel<1>, dim3(qp_blocks(pairs)), dim3(256), 0, stream, o, positions, cos_t, sin_t,
                                  table_rows, halves, out, dtype, nh, vd, P, pairs);
+    return rv_launch_status();
+}
+
+// A thread takes V neighbouring elements of a head.
+template <int V>
+__global__ void __launch_bounds__(256)
+gate_elements_kernel(const void* __restrict__ o, const float* __restrict__ logits, int g_stride, void* __restrict__ out, int dtype, int nh,
+                     int vd, int P, size_t total) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    const int per_head = vd / V, per_token = per_head * nh;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = i / per_token;
+        const int in_token = (int)(i - t * per_token), h = in_token / per_head, e = (in_token - h * per_head) * V;
+        float v[V], g[V];
+        qp_load_vec<V>(o, dtype, (t * nh + h) * P + e, v);
+        qp_load_vec<V>(logits, RV_DTYPE_F32, t * g_stride + (size_t)h * vd + e, g);
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] = v[j] / (1.0f + expf(-g[j]));
+        qp_store_vec<V>(out, dtype, (t * nh + h) * vd + e, v);
+    }
+}
+
+// logits: float rows of g_stride elements, of which the first nh * vd are the gates' (the pointer is at the first column).
+RV_EXPORT int rv_gate_elements(const void* o, const float* logits, int g_stride, void* out, int dtype, int n_tokens, int nh, int vd, int P,
+                               cudaStream_t stream) {
+    if (n_tokens < 0 || nh <= 0 || vd <= 0 || P < vd || g_stride < nh * vd) return RV_ERR_BAD_SIZE;
+    if (dtype & ~1) return RV_ERR_BAD_DTYPE;
+    if (n_tokens == 0) return RV_OK;
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(logits);
+    const size_t total = (size_t)n_tokens * nh * vd;
+    if (vd % 4 == 0 && P % 4 == 0 && g_stride % 4 == 0 && bits % 16 == 0)
+        RV_LAUNCH_ST = rv_launch(gate_elements_kernel<4>, dim3(qp_blocks(total / 4)), dim3(256), 0, stream, o, logits, g_stride, out, dtype,
+                                 nh, vd, P, total / 4);
+    else
+        RV_LAUNCH_ST = rv_launch(gate_elements_kernel<1>, dim3(qp_blocks(total)), dim3(256), 0, stream, o, logits, g_stride, out, dtype,
+                                 nh, vd, P, total);
     return rv_launch_status();
 }
 

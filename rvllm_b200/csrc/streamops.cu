@@ -17,6 +17,8 @@
 //   act_rows              relu(u)^2, optionally times one number per row, in the activations' type
 //   stream_combine        x += sum of up to three float32 terms, each with a factor, and up to two RMSNorms of the new x
 //                         from one row statistic (the inputs of sublayers that stand side by side)
+//   gated_combine         x += sum of up to two float32 terms, each times a vector and times sigmoid(logit + bias) element by element,
+//                         and an RMSNorm of the new x in groups of columns (the input of the next layer); without terms: the norm
 //   bigram_add            x + table[hash of (previous token, token)] as float32 (the start of a float32 stream); the last
 //                         token of a sequence's share is kept in its state row for the next step
 //
@@ -499,6 +501,155 @@ RV_EXPORT int rv_stream_combine(float* x, const float* y0, float c0, const float
         kernel = nv <= 1 ? stream_combine_kernel<1> : (nv <= 2 ? stream_combine_kernel<2> : (nv <= 4 ? stream_combine_kernel<4>
                                                                                                   : stream_combine_kernel<8>));
     RV_LAUNCH_ST = rv_launch(kernel, dim3(rows), dim3(threads), 0, stream, a);
+    return rv_launch_status();
+}
+
+// ------------------------------------------------------------------ stream += gated terms, and the norm in groups of the new stream
+struct GatedArgs {
+    float* x;
+    const float* y[2]; const float* scale[2]; int terms;
+    const void* gates; int gates_dtype, g_stride; const float* bias;     // logits [rows, g_stride], term k in columns k cols ..; bias alike
+    const void* gamma; int gamma_dtype; float eps; int groups;           // gamma null: no norm
+    void* out; int out_dtype;
+    int cols;
+};
+
+__device__ __forceinline__ float so_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float4 so_load4(const void* p, int dtype, size_t i) {          // four neighbours, i a multiple of 4
+    if (dtype == RV_DTYPE_F32) return *reinterpret_cast<const float4*>((const float*)p + i);
+    const uint2 u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
+// A row per block.  NV > 0: 4 columns a thread and access, the row in registers, every 32 accesses of a warp inside one group
+// (cols / 4 / groups a multiple of 32); NV = 0: any width and groups, the row is read again for the norm.
+template <int NV>
+__global__ void __launch_bounds__(256)
+gated_combine_kernel(const GatedArgs a) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    extern __shared__ float gc_smem[];
+    const size_t base = (size_t)blockIdx.x * a.cols, gbase = (size_t)blockIdx.x * a.g_stride;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    if constexpr (NV > 0) {
+        const int quads = a.cols / 4;
+        float4 v[NV];
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            if (i < quads) v[j] = reinterpret_cast<const float4*>(a.x + base)[i];
+        }
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            if (k >= a.terms) break;
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int i = threadIdx.x + j * blockDim.x;
+                if (i >= quads) continue;
+                const float4 y = reinterpret_cast<const float4*>(a.y[k] + base)[i];
+                const float4 s = reinterpret_cast<const float4*>(a.scale[k])[i];
+                const float4 b = reinterpret_cast<const float4*>(a.bias + (size_t)k * a.cols)[i];
+                const float4 g = so_load4(a.gates, a.gates_dtype, gbase + (size_t)k * a.cols + 4 * i);
+                v[j].x = fmaf(y.x * s.x, so_sigmoid(g.x + b.x), v[j].x);
+                v[j].y = fmaf(y.y * s.y, so_sigmoid(g.y + b.y), v[j].y);
+                v[j].z = fmaf(y.z * s.z, so_sigmoid(g.z + b.z), v[j].z);
+                v[j].w = fmaf(y.w * s.w, so_sigmoid(g.w + b.w), v[j].w);
+            }
+        }
+        if (a.terms) {
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int i = threadIdx.x + j * blockDim.x;
+                if (i < quads) reinterpret_cast<float4*>(a.x + base)[i] = v[j];
+            }
+        }
+        if (!a.gamma) return;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            float ss = i < quads ? v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w : 0.f;
+            ss = rv_warp_sum(ss);
+            if (lane == 0) gc_smem[j * warps + warp] = ss;               // one number per 128 columns
+        }
+        __syncthreads();
+        const int per = quads / a.groups / 32;
+        const float n = (float)(a.cols / a.groups);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            if (i >= quads) continue;                                    // (the same for the whole warp)
+            const int first = (j * warps + warp) / per * per;
+            float ss = 0.f;
+            for (int c = 0; c < per; ++c) ss += gc_smem[first + c];
+            const float r = 1.0f / sqrtf(ss / n + a.eps);
+            const float4 g = so_load4(a.gamma, a.gamma_dtype, 4 * (size_t)i);
+            const float o0 = v[j].x * r * g.x, o1 = v[j].y * r * g.y, o2 = v[j].z * r * g.z, o3 = v[j].w * r * g.w;
+            if (a.out_dtype == RV_DTYPE_F32) {
+                reinterpret_cast<float4*>((float*)a.out + base)[i] = make_float4(o0, o1, o2, o3);
+            } else {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(o0, o1), hi = __floats2bfloat162_rn(o2, o3);
+                uint2 pk;
+                pk.x = *reinterpret_cast<uint32_t*>(&lo); pk.y = *reinterpret_cast<uint32_t*>(&hi);
+                reinterpret_cast<uint2*>((__nv_bfloat16*)a.out + base)[i] = pk;
+            }
+        }
+    } else {
+        if (a.terms) {
+            for (int i = threadIdx.x; i < a.cols; i += blockDim.x) {
+                float v = a.x[base + i];
+#pragma unroll
+                for (int k = 0; k < 2; ++k)
+                    if (k < a.terms)
+                        v = fmaf(a.y[k][base + i] * a.scale[k][i],
+                                 so_sigmoid(so_load(a.gates, a.gates_dtype, gbase + (size_t)k * a.cols + i) + a.bias[(size_t)k * a.cols + i]), v);
+                a.x[base + i] = v;
+            }
+        }
+        if (!a.gamma) return;
+        __syncthreads();                                                 // the block's own writes of x are read across its threads
+        const int per = a.cols / a.groups;
+        for (int g = warp; g < a.groups; g += warps) {
+            float ss = 0.f;
+            for (int i = lane; i < per; i += 32) { const float v = a.x[base + (size_t)g * per + i]; ss = fmaf(v, v, ss); }
+            ss = rv_warp_sum(ss);
+            if (lane == 0) gc_smem[g] = 1.0f / sqrtf(ss / (float)per + a.eps);
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < a.cols; i += blockDim.x)
+            so_store(a.out, a.out_dtype, base + i, a.x[base + i] * gc_smem[i / per] * rv_load_param(a.gamma, a.gamma_dtype, i));
+    }
+}
+
+// y0, y1: float terms, the first null one ends them; scale0, scale1 float [cols]; gates [rows, g_stride] and bias float [terms * cols];
+// gamma null: no norm and no `out`.
+RV_EXPORT int rv_gated_combine(float* x, const float* y0, const float* scale0, const float* y1, const float* scale1, const void* gates,
+                               int gates_dtype, int g_stride, const float* bias, const void* gamma, int gamma_dtype, float eps, int groups,
+                               void* out, int out_dtype, int rows, int cols, cudaStream_t stream) {
+    if (rows < 0 || cols <= 0) return RV_ERR_BAD_SIZE;
+    if ((gates_dtype | gamma_dtype | out_dtype) & ~1) return RV_ERR_BAD_DTYPE;
+    const int terms = y0 ? (y1 ? 2 : 1) : 0;
+    if (terms && (!gates || !bias || !scale0 || (terms > 1 && !scale1) || g_stride < terms * cols)) return RV_ERR_BAD_SIZE;
+    if (gamma && (!out || groups <= 0 || cols % groups)) return RV_ERR_BAD_SIZE;
+    if (gamma && groups > 8192) return RV_ERR_UNSUPPORTED;
+    if (rows == 0 || (terms == 0 && !gamma)) return RV_OK;
+    const GatedArgs a = {x, {y0, y1}, {scale0, scale1}, terms, gates, gates_dtype, g_stride, bias, gamma, gamma_dtype, eps, groups, out,
+                         out_dtype, cols};
+    uintptr_t bits = reinterpret_cast<uintptr_t>(x);
+    if (terms) bits |= reinterpret_cast<uintptr_t>(y0) | reinterpret_cast<uintptr_t>(scale0) | reinterpret_cast<uintptr_t>(gates) | reinterpret_cast<uintptr_t>(bias);
+    if (terms > 1) bits |= reinterpret_cast<uintptr_t>(y1) | reinterpret_cast<uintptr_t>(scale1);
+    if (gamma) bits |= reinterpret_cast<uintptr_t>(gamma) | reinterpret_cast<uintptr_t>(out);
+    const int threads = cols >= 1024 ? 256 : 128;
+    const int nv = (cols / 4 + threads - 1) / threads;
+    auto kernel = gated_combine_kernel<0>;
+    size_t smem = (gamma ? groups : 1) * sizeof(float);
+    if (cols % 4 == 0 && g_stride % 4 == 0 && bits % 16 == 0 && nv <= 8 && (!gamma || (cols / 4) % (32 * groups) == 0)) {
+        kernel = nv <= 1 ? gated_combine_kernel<1> : (nv <= 2 ? gated_combine_kernel<2> : (nv <= 4 ? gated_combine_kernel<4>
+                                                                                                : gated_combine_kernel<8>));
+        smem = (size_t)8 * (threads / 32) * sizeof(float);
+    }
+    RV_LAUNCH_ST = rv_launch(kernel, dim3(rows), dim3(threads), smem, stream, a);
     return rv_launch_status();
 }
 

@@ -72,7 +72,8 @@ class Engine:
                     return t.to(self.dtype)
         else:
             source = WeightSource(model_dir)
-            source.check({n: ts.shape for n, ts in expected.items()}, self.spec.ignored_tensors)
+            source.check({n: ts.shape for n, ts in expected.items()}, self.spec.ignored_tensors,
+                         free={n: ts.free for n, ts in expected.items() if ts.free})
 
             def get(name: str) -> torch.Tensor:
                 return source.get(name, self.dtype, self.device)

@@ -288,22 +288,25 @@ class CudaKernels:
     # ------------------------------------------------------------------ attention
     def paged_attention(self, q, cache_layer, meta: AttentionMeta, num_heads, num_kv_heads, head_dim,
                         scale: float, window: Optional[int], softcap: Optional[float] = None,
-                        sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                        distance_bias=None) -> torch.Tensor:
         """Attention of the step's tokens over the paged cache (keys of this step included).
 
         `softcap`: scaled scores pass c * tanh(s / c); `sinks` (float [heads]): exp(sink) joins each head's
-        softmax denominator; `gate` (float [tokens, heads]): multiplies each head's output.
+        softmax denominator; `gate` (float [tokens, heads]): multiplies each head's output; `distance_bias` (a
+        `parts.distance.DistanceBias`): added to a score by the distance between query and key, after the cap.
 
         bfloat16 with a head size that is a multiple of 16 and pages of a power of two go to the
         tensor-core flash kernel (one token per sequence: the decode tiling, keys split over CTAs
         when the batch alone cannot fill the GPU); everything else goes to the plain kernel."""
         page = cache_layer.shape[3]
-        extras = softcap is not None or sinks is not None or gate is not None
+        extras = softcap is not None or sinks is not None or gate is not None or distance_bias is not None
         if q.dtype != torch.bfloat16 or head_dim % 16 or head_dim > 256 or (page & (page - 1)):
             return self.paged_attention_plain(q, cache_layer, meta, num_heads, num_kv_heads, head_dim, scale, window,
-                                              softcap, sinks, gate)
+                                              softcap, sinks, gate, distance_bias)
         self._check_attention_extras(q, num_heads, sinks, gate)
-        x = dict(softcap=softcap, sinks=sinks, gate=gate)
+        self._check_distance_bias(distance_bias, num_heads, num_kv_heads)
+        x = dict(softcap=softcap, sinks=sinks, gate=gate, distance_bias=distance_bias)
         out = torch.empty_like(q)
         group = num_heads // num_kv_heads
         # (the evenly cut decode kernel knows neither cap, sink nor gate: such layers stay with the split kernels)
@@ -332,7 +335,8 @@ class CudaKernels:
         return out
 
     def decode_attention(self, q, cache_layer, meta, out, num_heads, num_kv_heads, head_dim, scale, window,
-                         num_splits=1, q_filter=0, status=None, tma=None, early=None, softcap=None, sinks=None, gate=None):
+                         num_splits=1, q_filter=0, status=None, tma=None, early=None, softcap=None, sinks=None, gate=None,
+                         distance_bias=None):
         """Attention of the step's one-token sequences (all of them, or with q_filter 1 those among
         longer ones) with the decode tiling, the keys split over `num_splits` CTAs: the tiles come by
         TMA where the kernel is built for the sizes (head size 64 or 128, pages of 8 keys or more),
@@ -341,7 +345,7 @@ class CudaKernels:
         if not tma or head_dim not in (64, 128) or cache_layer.shape[3] < 8:
             return self.flash_attention(q, cache_layer, meta, out, num_heads, num_kv_heads, head_dim, scale, window,
                                         mode=1, num_splits=num_splits, q_filter=q_filter, max_q_len=1,
-                                        softcap=softcap, sinks=sinks, gate=gate)
+                                        softcap=softcap, sinks=sinks, gate=gate, distance_bias=distance_bias)
         _need(q, "q", torch.bfloat16, 2); _need(cache_layer, "cache_layer", torch.bfloat16, 5)
         lib = self._lib("attention_flash.cu", (f"-DHEAD_DIM={head_dim}",))
         T = q.shape[0]
@@ -354,7 +358,8 @@ class CudaKernels:
             _ptr(meta.ctx_lens), _ptr(out), _ptr(scratch), c_int(T), c_int(meta.num_seqs), c_int(num_heads), c_int(num_kv_heads),
             c_int(head_dim), c_int(cache_layer.shape[3]), c_int(meta.max_blocks), c_float(scale), c_int(window or 0), c_int(1),
             c_int(num_splits), c_int(q_filter), _ptr(status if status is not None else self._status),
-            c_int(1 if (early and self.pdl) else 0), c_float(softcap or 0.0), _ptr(sinks), _ptr(gate), self._stream())
+            c_int(1 if (early and self.pdl) else 0), c_float(softcap or 0.0), _ptr(sinks), _ptr(gate),
+            *self._distance_args(distance_bias), self._stream())
         _check("flash_decode_tma", st)
         return out
 
@@ -433,7 +438,8 @@ class CudaKernels:
         return out
 
     def flash_attention(self, q, cache_layer, meta, out, num_heads, num_kv_heads, head_dim, scale, window,
-                        mode=0, num_splits=1, q_filter=0, max_q_len=None, softcap=None, sinks=None, gate=None, value_dim=None):
+                        mode=0, num_splits=1, q_filter=0, max_q_len=None, softcap=None, sinks=None, gate=None, value_dim=None,
+                        distance_bias=None):
         """The mma.sync flash kernel (mode 0: 64 rows per CTA, prompt portions; mode 1: 16 rows, warps and CTAs split the keys).
         `value_dim`: the build for one-plane caches, whose rows are keys in full and values in their leading `value_dim`
         elements; `out` then has rows of that width."""
@@ -451,14 +457,14 @@ class CudaKernels:
             _ptr(out), _ptr(scratch), c_int(T), c_int(meta.num_seqs), c_int(num_heads), c_int(num_kv_heads),
             c_int(head_dim), c_int(cache_layer.shape[3]), c_int(meta.max_blocks), c_float(scale), c_int(window or 0),
             c_int(mode), c_int(max_q_len or meta.max_q_len), c_int(num_splits), c_int(q_filter), c_float(softcap or 0.0),
-            _ptr(sinks), _ptr(gate), self._stream())
+            _ptr(sinks), _ptr(gate), *self._distance_args(distance_bias), self._stream())
         _check("flash_attention", st)
         if num_splits > 1:
             COUNTERS['launches'] += 1
         return out
 
     def attention_tcgen05(self, q, cache_layer, meta, out, num_heads, num_kv_heads, head_dim, scale, window, status=None,
-                          softcap=None, sinks=None, gate=None, value_dim=None):
+                          softcap=None, sinks=None, gate=None, value_dim=None, distance_bias=None):
         """The tcgen05 flash-attention kernel for the sequences of a step that bring more than one
         token (bfloat16, head size 64 or 128, groups of up to 128 heads, pages of at least 8 keys).
         `value_dim`: the build for one-plane caches (rows of `head_dim` elements, up to 256, that are keys in full and
@@ -473,20 +479,22 @@ class CudaKernels:
             _ptr(meta.cu_seqlens), _ptr(meta.ctx_lens), _ptr(out), c_int(q.shape[0]), c_int(meta.num_seqs),
             c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(cache_layer.shape[3]), c_int(meta.max_blocks),
             c_float(scale), c_int(window or 0), c_int(meta.max_q_len), _ptr(status if status is not None else self._status),
-            c_float(softcap or 0.0), _ptr(sinks), _ptr(gate), self._stream())
+            c_float(softcap or 0.0), _ptr(sinks), _ptr(gate), *self._distance_args(distance_bias), self._stream())
         _check("attention_tcgen05", st)
         return out
 
     def paged_attention_plain(self, q, cache_layer, meta, num_heads, num_kv_heads, head_dim, scale, window,
-                              softcap=None, sinks=None, gate=None):
+                              softcap=None, sinks=None, gate=None, distance_bias=None):
         _need(q, "q", dims=2); _need(cache_layer, "cache_layer", q.dtype, 5)
         self._check_attention_extras(q, num_heads, sinks, gate)
+        self._check_distance_bias(distance_bias, num_heads, num_kv_heads)
         out = torch.empty_like(q)
         st = self._lib("attention_ref.cu").rv_paged_attention_ref_ex(
             _ptr(q), _ptr(cache_layer), _ptr(meta.block_tables), _ptr(meta.cu_seqlens), _ptr(meta.ctx_lens),
             _ptr(meta.token_seq), _ptr(out), c_int(q.shape[0]), c_int(num_heads), c_int(num_kv_heads),
             c_int(head_dim), c_int(cache_layer.shape[3]), c_int(meta.max_blocks), c_float(scale), c_int(window or 0),
-            c_float(softcap or 0.0), _ptr(sinks), _ptr(gate), c_int(2), c_int(head_dim), c_int(self._dt(q, "q")), self._stream())
+            c_float(softcap or 0.0), _ptr(sinks), _ptr(gate), c_int(2), c_int(head_dim), c_int(self._dt(q, "q")),
+            *self._distance_args(distance_bias, natural=True), self._stream())
         _check("paged_attention_plain", st)
         return out
 
@@ -500,6 +508,22 @@ class CudaKernels:
             _need(gate, "gate", torch.float32, 2)
             if tuple(gate.shape) != (q.shape[0], num_heads):
                 raise KernelError(f"attention: gate of shape {tuple(gate.shape)} for {q.shape[0]} tokens of {num_heads} heads")
+
+    @staticmethod
+    def _distance_args(distance_bias, natural: bool = False):
+        """(table, distances) for a kernel that works in powers of two, or - `natural` - in powers of e."""
+        if distance_bias is None:
+            return _ptr(None), c_int(0)
+        return _ptr(distance_bias.natural if natural else distance_bias.log2), c_int(distance_bias.distances)
+
+    @staticmethod
+    def _check_distance_bias(distance_bias, num_heads, num_kv_heads):
+        if distance_bias is None:
+            return
+        for t in (distance_bias.natural, distance_bias.log2):
+            _need(t, "distance bias", torch.float32, 3)
+            if t.shape[0] != num_kv_heads or t.shape[1] < 1 or t.shape[2] * num_kv_heads != num_heads or t.shape != distance_bias.natural.shape:
+                raise KernelError(f"attention: a distance bias of shape {tuple(t.shape)} for {num_heads} heads on {num_kv_heads} key/value heads")
 
     # ------------------------------------------------------------------ linear layers
     def linear(self, x, weight, bias=None, residual=None, out_dtype=None, norm=None) -> torch.Tensor:
@@ -1337,6 +1361,59 @@ class CudaKernels:
         _check("latent_prepare", st)
         return q_plain, q_row, gate
 
+    def _latent_tables(self, what: str, cos, sin, rot_dim: int):
+        if cos is None:
+            return 0, 1
+        _need(cos, "cos", torch.float32, 2); _need(sin, "sin", torch.float32, 2)
+        if not 0 < 2 * cos.shape[1] <= rot_dim or sin.shape != cos.shape:
+            raise KernelError(f"{what}: cos/sin tables must be [rows, dims/2] with dims <= {rot_dim}")
+        return 2 * cos.shape[1], cos.shape[0]
+
+    def latent_down(self, proj, q_gamma, c_gamma, eps: float, positions, cos, sin, slot_mapping, cache_layer, q_rank: int, rot_dim: int,
+                    kv_rank: int, out_dtype, heads: int = 0, write_kv: bool = True, halves: bool = False):
+        """What `latent_prepare` does to the latent and the shared key part, for queries with a low-rank row of their own: proj rows
+        [cq': q_rank | c': kv_rank | r: rot_dim | gate logits: heads].  Returns (cq' RMS-normalised with weight `q_gamma`
+        [T, q_rank], sigmoid(gate logits) float [T, heads] or None)."""
+        _need(proj, "proj", dims=2); _need(positions, "positions", torch.int32, 1)
+        _need(q_gamma, "q_gamma", dims=1); _need(c_gamma, "c_gamma", dims=1)
+        T, row = proj.shape[0], kv_rank + rot_dim
+        if proj.shape[1] != q_rank + row + heads or q_gamma.shape[0] != q_rank or c_gamma.shape[0] != kv_rank:
+            raise KernelError(f"latent_down: rows of {proj.shape[1]} columns do not fit latents of {q_rank} and {kv_rank} + {rot_dim}"
+                              + (f" and {heads} gates" if heads else ""))
+        rot, table_rows = self._latent_tables("latent_down", cos, sin, rot_dim)
+        if write_kv:
+            _need(cache_layer, "cache_layer", out_dtype, 5); _need(slot_mapping, "slot_mapping", torch.int32, 1)
+            if tuple(cache_layer.shape[1:3]) != (1, 1) or cache_layer.shape[4] != row:
+                raise KernelError(f"latent_down: cache layer of shape {tuple(cache_layer.shape)} does not hold one row of {row} per token")
+        low = torch.empty((T, q_rank), dtype=out_dtype, device=proj.device)
+        gate = torch.empty((T, heads), dtype=torch.float32, device=proj.device) if heads else None
+        st = self._lib("latent.cu").rv_latent_down(
+            _ptr(proj), c_int(self._dt(proj, "proj")), c_int(proj.shape[1]), _ptr(q_gamma), c_int(self._dt(q_gamma, "q_gamma")),
+            _ptr(c_gamma), c_int(self._dt(c_gamma, "c_gamma")), _ptr(positions), _ptr(cos), _ptr(sin), c_int(rot), c_int(table_rows),
+            _ptr(slot_mapping if write_kv else None), _ptr(cache_layer if write_kv else None), _ptr(low), c_int(_DT[out_dtype]), _ptr(gate),
+            c_int(T), c_int(heads), c_int(q_rank), c_int(rot_dim), c_int(kv_rank), c_float(eps), c_int(1 if write_kv else 0),
+            c_int(1 if halves else 0), self._stream())
+        _check("latent_down", st)
+        return low, gate
+
+    def latent_queries(self, q, positions, cos, sin, num_heads: int, head_dim: int, rot_dim: int, kv_rank: int, out_dtype,
+                       halves: bool = False):
+        """The queries' part of `latent_prepare` alone: q rows [heads x (head_dim + rot_dim)] -> (q_plain [T, heads, head_dim],
+        q_row [T, heads, kv_rank + rot_dim] with its last rot_dim columns filled)."""
+        _need(q, "q", dims=2); _need(positions, "positions", torch.int32, 1)
+        T = q.shape[0]
+        if q.shape[1] != num_heads * (head_dim + rot_dim):
+            raise KernelError(f"latent_queries: rows of {q.shape[1]} columns for {num_heads} heads of {head_dim} + {rot_dim}")
+        rot, table_rows = self._latent_tables("latent_queries", cos, sin, rot_dim)
+        q_plain = torch.empty((T, num_heads, head_dim), dtype=out_dtype, device=q.device)
+        q_row = torch.empty((T, num_heads, kv_rank + rot_dim), dtype=out_dtype, device=q.device)
+        st = self._lib("latent.cu").rv_latent_queries(
+            _ptr(q), c_int(self._dt(q, "q")), _ptr(positions), _ptr(cos), _ptr(sin), c_int(rot), c_int(table_rows), _ptr(q_plain),
+            _ptr(q_row), c_int(_DT[out_dtype]), c_int(T), c_int(num_heads), c_int(head_dim), c_int(rot_dim), c_int(kv_rank),
+            c_int(1 if halves else 0), self._stream())
+        _check("latent_queries", st)
+        return q_plain, q_row
+
     def head_linear(self, x, weight, out: Optional[torch.Tensor] = None, out_dtype=None) -> torch.Tensor:
         """out[t, h, :] = weight[h] x[t, h, :] for x [T, heads, K], weight [heads, N, K]; float accumulation.  x and out may be
         slices of wider rows (their last dimension contiguous); without `out` a new [T, heads, N] tensor is returned."""
@@ -1446,19 +1523,20 @@ class CudaKernels:
             _ptr(q_row), _ptr(cache_layer), _ptr(meta.block_tables), _ptr(meta.cu_seqlens), _ptr(meta.ctx_lens),
             _ptr(meta.token_seq), _ptr(out), c_int(T), c_int(num_heads), c_int(1), c_int(row), c_int(cache_layer.shape[3]),
             c_int(meta.max_blocks), c_float(scale), c_int(0), c_float(0.0), _ptr(sinks), _ptr(gate), c_int(1), c_int(value_dim),
-            c_int(self._dt(q_row, "q_row")), self._stream())
+            c_int(self._dt(q_row, "q_row")), *self._distance_args(None), self._stream())
         _check("latent_attention", st)
         return out
 
     # ------------------------------------------------------------------ mixture of experts
     def moe_experts(self, x, chosen, gate_up, down, weight: float, add: Optional[torch.Tensor] = None, out_dtype=None,
                     weights: Optional[torch.Tensor] = None, activation: str = "silu",
-                    add_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    add_scale: Optional[torch.Tensor] = None, identity: bool = False) -> torch.Tensor:
         """out[t] = (add_scale[t] * add[t]) + weight * sum_k weights[t, k] down[e] a_e(x_t), e = chosen[t, k].
         activation "silu": gated experts, a_e(x) = silu(gate[e] x) * (up[e] x), gate_up [experts, 2 ff, width] (gate rows, then up
         rows); "relu2": plain experts, a_e(x) = relu(up[e] x)^2, `gate_up` is up [experts, ff, width].  down [experts, width, ff],
         chosen int32 [T, top], weights float32 [T, top] or None (all 1), add float32 [T, width] or None,
-        add_scale float32 [T] or None (all 1)."""
+        add_scale float32 [T] or None (all 1).  Numbers outside 0 .. experts - 1 contribute nothing - or, with `identity`, numbers
+        from `experts` on contribute x_t itself."""
         _need(x, "x", dims=2); _need(chosen, "chosen", torch.int32, 2)
         _need(gate_up, "gate_up", x.dtype, 3); _need(down, "down", x.dtype, 3)
         if activation not in ("silu", "relu2"):
@@ -1486,13 +1564,13 @@ class CudaKernels:
         if out_dtype not in (x.dtype, torch.float32):
             raise KernelError(f"moe_experts: result type {out_dtype} for operands of {x.dtype}")
         if x.dtype == torch.bfloat16 and T >= self.MOE_GROUPED_MIN_TOKENS and width % 8 == 0 and ff % 8 == 0 and E <= 4096:
-            return self._moe_grouped(x, chosen, gate_up, down, weight, add, out_dtype, weights, gated, add_scale)
+            return self._moe_grouped(x, chosen, gate_up, down, weight, add, out_dtype, weights, gated, add_scale, identity)
         act = torch.empty((T * top, ff), dtype=x.dtype, device=x.device)
         out = torch.empty((T, width), dtype=out_dtype, device=x.device)
         st = self._lib("moe.cu").rv_moe_experts_ex(
             _ptr(x), _ptr(chosen), _ptr(weights), _ptr(gate_up), _ptr(down), _ptr(act), _ptr(add), _ptr(add_scale),
             _ptr(out), c_int(1 if out_dtype == torch.float32 else 0), c_int(T), c_int(top), c_int(E), c_int(ff), c_int(width), c_float(weight),
-            c_int(1 if gated else 0), c_int(self._dt(x, "x")), self._stream())
+            c_int(1 if gated else 0), c_int(1 if identity else 0), c_int(self._dt(x, "x")), self._stream())
         _check("moe_experts", st)
         COUNTERS['launches'] += 1
         return out
@@ -1500,7 +1578,8 @@ class CudaKernels:
     MOE_GROUPED_MIN_TOKENS = 128      # tokens of a step from which the experts' products run grouped on the tcgen05 GEMM ...
     MOE_GROUPED_PAIRS = True          # ... on pairs of CTAs (cta_group::2): two blocks of 128 rows of one expert share every tile of its weights
 
-    def _moe_grouped(self, x, chosen, gate_up, down, weight, add, out_dtype, weights=None, gated=True, add_scale=None):
+    def _moe_grouped(self, x, chosen, gate_up, down, weight, add, out_dtype, weights=None, gated=True, add_scale=None,
+                     identity=False):
         """`moe_experts` for many bfloat16 tokens: the (token, slot) pairs sorted by expert, every expert's rows padded to
         whole blocks of 128, two grouped tcgen05 products over the sorted rows (gate/up with the SiLU epilogue - plain experts:
         up with the squared relu in its epilogue - then down with a float32 result), and the weighted sum per token.  Everything is decided on the device; the buffers are sized for the worst case (every
@@ -1540,18 +1619,23 @@ class CudaKernels:
         out = torch.empty((T, width), dtype=out_dtype, device=dev)
         _check("moe_combine", moe.rv_moe_combine(_ptr(ys), _ptr(row_of), _ptr(add), _ptr(out), c_int(1 if out_dtype == torch.float32 else 0),
                                                  c_int(T), c_int(top), c_int(width), c_float(weight), _ptr(weights), _ptr(add_scale),
-                                                 self._stream()))
+                                                 _ptr(x if identity else None), _ptr(chosen), c_int(E), self._stream()))
         return out
 
     def moe_route_top(self, scores, correction, experts: int, top: int, groups: int, keep: int, weight_eps: float,
-                      shared_gate: bool = False, scoring: str = "sigmoid"):
+                      shared_gate: bool = False, scoring: str = "sigmoid", group_score: str = "top2"):
         """A router's choice from its float32 logits [T, experts (+ 1)]: s = sigmoid(logits); the `top` experts with the largest
         s + correction among those of the `keep` best of `groups` equal groups of neighbouring experts (a group counts by the
         sum of its two largest corrected scores).  Returns (chosen int32 [T, top], weights float32 [T, top] = the chosen s over
         their sum + weight_eps, sigmoid of the last column float32 [T] with `shared_gate`, else None).  scoring "softmax": the choice
-        is made among logits + correction, and the weights are the softmax over the chosen ones (then divided by 1 + weight_eps / sum)."""
-        if scoring not in ("sigmoid", "softmax"):
-            raise KernelError(f"moe_route_top: scoring {scoring!r} is not known (sigmoid, softmax)")
+        is made among logits + correction, and the weights are the softmax over the chosen ones (then divided by 1 + weight_eps / sum).
+        scoring "softmax_all": s = softmax(logits) over all experts, otherwise as "sigmoid".  group_score "max": a group counts by
+        its largest corrected score alone."""
+        modes = {"sigmoid": 0, "softmax": 1, "softmax_all": 2}
+        if scoring not in modes:
+            raise KernelError(f"moe_route_top: scoring {scoring!r} is not known ({', '.join(modes)})")
+        if group_score not in ("top2", "max"):
+            raise KernelError(f"moe_route_top: group score {group_score!r} is not known (top2, max)")
         _need(scores, "scores", torch.float32, 2); _need(correction, "correction", torch.float32, 1)
         T = scores.shape[0]
         if scores.shape[1] != experts + (1 if shared_gate else 0) or correction.shape[0] != experts:
@@ -1561,7 +1645,8 @@ class CudaKernels:
         gate = torch.empty((T,), dtype=torch.float32, device=scores.device) if shared_gate else None
         st = self._lib("moe.cu").rv_moe_route_top(
             _ptr(scores), c_int(scores.shape[1]), _ptr(correction), _ptr(chosen), _ptr(weights), _ptr(gate), c_int(T), c_int(experts),
-            c_int(top), c_int(groups), c_int(keep), c_float(weight_eps), c_int(1 if scoring == "softmax" else 0), self._stream())
+            c_int(top), c_int(groups), c_int(keep), c_float(weight_eps), c_int(modes[scoring]),
+            c_int(1 if group_score == "max" else 0), self._stream())
         _check("moe_route_top", st)
         return chosen, weights, gate
 
@@ -1627,7 +1712,8 @@ class CudaKernels:
     # ------------------------------------------------------------------ unit-norm attention, mLSTM
     def qk_prepare(self, proj, positions, cos, sin, slot_mapping, cache_layer, num_heads: int, num_kv_heads: int, head_dim: int,
                    value_dim: int, slot_dim: int, out_dtype, eps: Optional[float] = None, halves: bool = False, with_gate: bool = False,
-                   write_kv: bool = True, maps: int = 1, bias: Optional[torch.Tensor] = None, value_tables=None):
+                   write_kv: bool = True, maps: int = 1, bias: Optional[torch.Tensor] = None, value_tables=None, norms=None,
+                   temperature=None, keep_values: Optional[torch.Tensor] = None, mix_values=None):
         """proj float32 rows [q: heads x maps x head_dim | k: kv heads x maps x head_dim | v: kv heads x value_dim | gate logits:
         heads] (k and v only with `write_kv`), plus `bias` (float32, a number per column of q, k and v).  q and k: the leading
         2 * cos.shape[1] elements of every map turn in pairs (2i, 2i + 1) - with `halves`: (i, i + cos.shape[1]) -, then, with
@@ -1635,8 +1721,15 @@ class CudaKernels:
         all its elements.  k (its maps side by side) and v go into the token's cache slot, in heads of `slot_dim` elements
         whose tail is zeros; a query row of map m holds its elements at m * head_dim and zeros elsewhere, so that its product
         with the key row is map m's score.  Returns (q [T, heads * maps * slot_dim] in `out_dtype`, sigmoid(gate logits)
-        float32 [T, heads] or None)."""
-        _need(proj, "proj", torch.float32, 2); _need(positions, "positions", torch.int32, 1)
+        float32 [T, heads] or None).
+
+        norms = (q gamma, k gamma), float32 [head_dim] each: instead of the unit norm, x / sqrt(mean(x^2) + eps) * gamma in FRONT
+        of the rotation.  temperature = (c, every): a query at position p is multiplied by 1 + c ln(floor((p + 1) / every) + 1).
+        keep_values (float32 [T, kv heads * value_dim]) receives the values as projected, with their biases; mix_values =
+        (such a tensor, l): the value becomes (1 - l) v + l times it.  proj may be the leading columns of a wider matrix."""
+        if proj.dim() != 2 or proj.dtype != torch.float32 or not proj.is_cuda or proj.stride(1) != 1:
+            raise KernelError(f"proj must be float32 rows on the device, got {proj.dtype} {tuple(proj.shape)} with strides {proj.stride()}")
+        _need(positions, "positions", torch.int32, 1)
         T = proj.shape[0]
         cols = maps * num_heads * head_dim + (num_kv_heads * (maps * head_dim + value_dim) if write_kv else 0)
         if proj.shape[1] != cols + (num_heads if with_gate else 0) or slot_dim < max(maps * head_dim, value_dim):
@@ -1658,6 +1751,19 @@ class CudaKernels:
             _need(bias, "bias", torch.float32, 1)
             if bias.shape[0] != cols:
                 raise KernelError(f"qk_prepare: {bias.shape[0]} biases for {cols} columns")
+        q_gamma, k_gamma = norms if norms is not None else (None, None)
+        if norms is not None:
+            for g in norms:
+                _need(g, "norm weight", torch.float32, 1)
+                if g.shape[0] != head_dim or eps is None:
+                    raise KernelError(f"qk_prepare: a norm weight of {g.shape[0]} (eps {eps}) for heads of {head_dim}")
+        first, lam = mix_values if mix_values is not None else (None, 0.0)
+        for v in (keep_values, first):
+            if v is not None:
+                _need(v, "values", torch.float32, 2)
+                if tuple(v.shape) != (T, num_kv_heads * value_dim) or not write_kv:
+                    raise KernelError(f"qk_prepare: kept values of shape {tuple(v.shape)} for {T} tokens of {num_kv_heads} x {value_dim}")
+        coef, every = temperature if temperature is not None else (0.0, 0)
         page = 1
         if write_kv:
             _need(cache_layer, "cache_layer", out_dtype, 5); _need(slot_mapping, "slot_mapping", torch.int32, 1)
@@ -1666,12 +1772,13 @@ class CudaKernels:
             page = cache_layer.shape[3]
         q = torch.empty((T, num_heads * maps * slot_dim), dtype=out_dtype, device=proj.device)
         gate = torch.empty((T, num_heads), dtype=torch.float32, device=proj.device) if with_gate else None
-        st = self._lib("qk_prepare.cu").rv_qk_prepare(
-            _ptr(proj), c_int(proj.shape[1]), _ptr(bias), _ptr(positions), _ptr(cos), _ptr(sin), c_int(rot), c_int(table_rows),
+        st = self._lib("qk_prepare.cu").rv_qk_prepare_ex(
+            _ptr(proj), c_int(proj.stride(0) if T > 1 else max(proj.stride(0), proj.shape[1])), _ptr(bias), _ptr(positions), _ptr(cos), _ptr(sin), c_int(rot), c_int(table_rows),
             c_int(1 if halves else 0), _ptr(vcos), _ptr(vsin), c_int(vcos.shape[0] if vcos is not None else 1),
             _ptr(slot_mapping if write_kv else None), _ptr(cache_layer if write_kv else None), _ptr(q), c_int(_DT[out_dtype]), _ptr(gate),
             c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(value_dim), c_int(slot_dim), c_int(maps), c_int(page),
-            c_float(eps or 0.0), c_int(1 if eps is not None else 0), c_int(1 if write_kv else 0), self._stream())
+            c_float(eps or 0.0), c_int(1 if eps is not None and norms is None else 0), c_int(1 if write_kv else 0), _ptr(q_gamma),
+            _ptr(k_gamma), c_float(coef), c_int(every), _ptr(keep_values), _ptr(first), c_float(lam), self._stream())
         _check("qk_prepare", st)
         return q, gate
 
@@ -1696,6 +1803,21 @@ class CudaKernels:
             _ptr(o), _ptr(positions), _ptr(cos), _ptr(sin), c_int(cos.shape[0]), c_int(1 if halves else 0), _ptr(out), c_int(self._dt(o, "o")),
             c_int(T), c_int(heads), c_int(value_dim), c_int(slot_dim), self._stream())
         _check("turn_back", st)
+        return out
+
+    def gate_elements(self, o, proj, col0: int, heads: int, value_dim: int, slot_dim: int) -> torch.Tensor:
+        """The leading `value_dim` elements of every head of o [T, heads * slot_dim], each times the sigmoid of its own logit, which
+        lie in the columns from `col0` on of the float32 rows `proj`.  Returns [T, heads * value_dim]."""
+        _need(o, "o", dims=2); _need(proj, "proj", torch.float32, 2)
+        T = o.shape[0]
+        if o.shape[1] != heads * slot_dim or slot_dim < value_dim or proj.shape[0] != T or not 0 <= col0 <= proj.shape[1] - heads * value_dim:
+            raise KernelError(f"gate_elements: rows of {o.shape[1]} and {proj.shape[1]} (from {col0} on) for {heads} heads of {value_dim} "
+                              f"in slots of {slot_dim}")
+        out = torch.empty((T, heads * value_dim), dtype=o.dtype, device=o.device)
+        st = self._lib("qk_prepare.cu").rv_gate_elements(_ptr(o), c_void_p(proj.data_ptr() + 4 * col0), c_int(proj.shape[1]), _ptr(out),
+                                                         c_int(self._dt(o, "o")), c_int(T), c_int(heads), c_int(value_dim), c_int(slot_dim),
+                                                         self._stream())
+        _check("gate_elements", st)
         return out
 
     def map_difference(self, o, lam: float, eps: float, factor: float, heads: int, value_dim: int, slot_dim: int) -> torch.Tensor:
@@ -1743,6 +1865,45 @@ class CudaKernels:
                                                          self._stream())
         _check("stream_combine", st)
         return x, outs
+
+    def gated_combine(self, x, terms, scales, gates, bias, norm, out_dtype):
+        """x += sum over k of terms[k] * scales[k] * sigmoid(gates[:, k cols : (k + 1) cols] + bias[k cols : (k + 1) cols]) on the
+        float32 stream, in place (up to two float32 terms); then, with norm = (gamma, eps, groups), the new x under an RMSNorm in
+        `groups` equal parts of its columns, in `out_dtype`.  Returns (x, normed x or None)."""
+        _need(x, "x", torch.float32, 2)
+        rows, cols = x.shape
+        n = len(terms)
+        if n > 2 or len(scales) != n:
+            raise KernelError(f"gated_combine: {n} terms (at most two) and {len(scales)} vectors")
+        for y, s in zip(terms, scales):
+            _need(y, "term", torch.float32, 2); _need(s, "scale", torch.float32, 1)
+            if y.shape != x.shape or s.shape[0] != cols:
+                raise KernelError(f"gated_combine: {tuple(y.shape)} times {s.shape[0]} added to {tuple(x.shape)}")
+        if n:
+            _need(gates, "gates", dims=2); _need(bias, "bias", torch.float32, 1)
+            if tuple(gates.shape) != (rows, n * cols) or bias.shape[0] != n * cols:
+                raise KernelError(f"gated_combine: gates {tuple(gates.shape)} and {bias.shape[0]} biases for {n} terms of {tuple(x.shape)}")
+        gamma, eps, groups = norm if norm is not None else (None, 0.0, 1)
+        out = None
+        if gamma is not None:
+            _need(gamma, "gamma", dims=1)
+            if gamma.shape[0] != cols or groups < 1 or cols % groups:
+                raise KernelError(f"gated_combine: gamma of {gamma.shape[0]} in {groups} groups for rows of {cols}")
+            out = torch.empty((rows, cols), dtype=out_dtype, device=x.device)
+        y = list(terms) + [None] * (2 - n)
+        s = list(scales) + [None] * (2 - n)
+        st = self._lib("streamops.cu").rv_gated_combine(
+            _ptr(x), _ptr(y[0]), _ptr(s[0]), _ptr(y[1]), _ptr(s[1]), _ptr(gates if n else None),
+            c_int(self._dt(gates, "gates") if n else 0), c_int(n * cols), _ptr(bias if n else None), _ptr(gamma),
+            c_int(self._dt(gamma, "gamma") if gamma is not None else 0), c_float(eps), c_int(groups), _ptr(out),
+            c_int(_DT[out_dtype] if out is not None else 0), c_int(rows), c_int(cols), self._stream())
+        _check("gated_combine", st)
+        return x, out
+
+    def grouped_rmsnorm(self, x, gamma, eps: float, groups: int, out_dtype=None) -> torch.Tensor:
+        """x / sqrt(mean(part^2) + eps) * gamma, the row in `groups` equal parts with a statistic each."""
+        xf = x if x.dtype == torch.float32 else x.float()
+        return self.gated_combine(xf, [], [], None, None, (gamma, eps, groups), out_dtype or x.dtype)[1]
 
     def mingru(self, proj, z_bias, x_bias, cu_seqlens, state_slots, state, width: int, single: bool, out_dtype) -> torch.Tensor:
         """The minGRU recurrence over the step's tokens: proj float32 rows [Z | X | G] of `width` columns each;

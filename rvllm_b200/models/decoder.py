@@ -54,7 +54,10 @@ class _Layer:
 
     def named_parts(self):
         n = self.spec.names
-        return [(self.spec.prefix + n.get(role, role + "."), part) for role, part in self.parts.items()]
+        named = [(self.spec.prefix + n.get(role, role + "."), part) for role, part in self.parts.items()]
+        if hasattr(self.block, "tensor_specs"):          # an arrangement with tensors of its own
+            named.append((self.spec.prefix, self.block))
+        return named
 
 
 class DecoderModel:

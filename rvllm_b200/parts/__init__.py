@@ -1,12 +1,12 @@
 from .base import (Part, TensorSpec, KvCacheNeed, StateNeed, CompositeNeed, Registry, MIXERS, FEED_FORWARDS, NORMS,
                    POSITION_ENCODINGS, BLOCKS, HOOKS, FAMILIES)
 from .linear import Linear
-from .norm import RMSNorm, DynamicTanh
+from .norm import RMSNorm, GroupedRMSNorm, DynamicTanh
 from .rope import RotaryEncoding, inverse_frequencies
 from .attention import PagedAttention
 from .mlp import GatedMLP, ClampedGluMLP
 from .block import (PreNormResidualBlock, OutputNormResidualBlock, SandwichNormResidualBlock,
-                    PreNormStreamResidualBlock, SideBySideResidualBlock)
+                    PreNormStreamResidualBlock, SideBySideResidualBlock, SharedNormGatedResidualBlock)
 from .sink_attention import GatedSinkAttention
 from .mamba2 import Mamba2Mixer
 from .latent_attention import LatentAttention
@@ -22,3 +22,5 @@ from .unit_attention import UnitQkAttention
 from .mlstm import MLstmMixer
 from .differential_attention import DifferentialAttention
 from .min_gru import MinGruMixer
+from .distance import DistanceBias, distance_table
+from .normed_attention import NormedQkAttention

@@ -15,8 +15,9 @@ tensors it owns (`tensor_specs`, names relative to its prefix) and receives them
 * feed-forward: `__call__(x, ctx, residual)` -> residual + f(x).
 * block: built from `parts`, the layer's built parts by role name (which roles it needs is the
   block's own matter), plus its parameters; `__call__(x, ctx, cache, write_cache)` -> x.  A block whose input is the
-  stream under RMSNorms may offer `input_norms()` -> [(gamma, eps), ...]: the block that runs before it can then form them in the
-  kernel that writes the stream (`ctx.following_norms`, None where something else stands between).
+  stream under RMSNorms may offer `input_norms()` -> [(gamma, eps), ...] - (gamma, eps, groups) for a norm in groups -: the block that
+  runs before it can then form them in the kernel that writes the stream (`ctx.following_norms`, None where something else
+  stands between).  A block with tensors of its own offers `tensor_specs()` and `bind(get)`, as a part does; they lie below the layer's prefix.
 * hook: `__call__(x, ctx)` -> x, on the embedded tokens or on the float32 logits.  A hook on the embedded tokens that
   keeps something per sequence offers `cache_need()`; it is then called `(x, ctx, cache)` with a cache slot of its own.
 
@@ -39,6 +40,7 @@ import torch
 class TensorSpec:
     shape: Tuple[int, ...]
     init: str          # "matrix", "norm" or "bias": which random distribution fills it
+    free: Tuple[int, ...] = ()     # dimensions whose size the checkpoint decides (`shape` then says what a random tensor has)
 
 
 @dataclass(frozen=True)

@@ -12,7 +12,8 @@ from __future__ import annotations
 
 import torch
 
-from .base import BLOCKS
+from .base import BLOCKS, Part, TensorSpec
+from .linear import Linear
 
 
 class PreNormResidualBlock:
@@ -254,7 +255,7 @@ class SideBySideResidualBlock:
             x, _ = k.stream_combine(x, terms[:3], [], dtype)
             terms = terms[3:]
         following = ctx.following_norms
-        if following is not None and len(following) > 2:
+        if following is not None and (len(following) > 2 or any(len(n) != 2 for n in following)):     # (not norms this kernel forms)
             following = None
         x, normed = k.stream_combine(x, terms, following or [], dtype)
         if following:
@@ -263,3 +264,70 @@ class SideBySideResidualBlock:
 
 
 BLOCKS.register("side_by_side_residual", SideBySideResidualBlock)
+
+
+class SharedNormGatedResidualBlock(Part):
+    """`shared_norm_gated_residual`: with h = norm(x),
+
+        x + s1 sigmoid(W1 h + b1) mixer(h) + s2 sigmoid(W2 h + b2) feed_forward(h)        element by element
+
+    One norm (an RMSNorm in groups), whose output both sublayers and both gates read; s1 and s2 are learned vectors.  A layer
+    may have no feed-forward (and then no s2, W2, b2).
+
+    The stream x is float32 whatever the engine's type (`ModelSpec.residual_dtype`).  Both gates are one stacked product; the
+    sublayers return float32, and one kernel forms the sigmoids, adds both terms to the stream and, where the next block of the
+    run order offers its `input_norms`, leaves that block's input as well.  It travels beside the stream in `ctx.extras`; a block
+    that finds none (the first layer) forms it.  Tensors below the layer's prefix: ls1, rg1, rg1.b (ls2, rg2, rg2.b)."""
+    ROLES = ("mixer", "norm")
+    OPTIONAL = ("feed_forward",)
+    KEY = "shared_normed_stream"
+
+    def __init__(self, parts, hidden_size: int, scale: str = "ls", gate: str = "rg", suffix: str = "", bias_suffix: str = ".b"):
+        from ..errors import ConfigError
+        names = set(parts)
+        if not set(self.ROLES) <= names or not names <= set(self.ROLES + self.OPTIONAL):
+            raise ConfigError(f"the shared-norm gated residual block arranges {', '.join(self.ROLES)} and optionally "
+                              f"{', '.join(self.OPTIONAL)}; got {', '.join(sorted(parts))}")
+        self.mixer, self.norm, self.feed_forward = parts["mixer"], parts["norm"], parts.get("feed_forward")
+        if not hasattr(self.norm, "as_grouped"):
+            raise ConfigError("the shared-norm gated residual block needs a norm that offers `as_grouped()` (an RMSNorm in groups)")
+        self.hidden_size = hidden_size
+        numbers = ("1",) if self.feed_forward is None else ("1", "2")
+        self.scale_names = [scale + n for n in numbers]
+        self.gates = Linear(hidden_size, [hidden_size] * len(numbers), [gate + n for n in numbers], bias=True, suffix=suffix,
+                            bias_suffix=bias_suffix)
+        self.scales = []
+        self.gate_bias = None
+
+    def tensor_specs(self):
+        return {**self.gates.tensor_specs(), **{n: TensorSpec((self.hidden_size,), "norm") for n in self.scale_names}}
+
+    def bind(self, get):
+        self.gates.bind(get)
+        self.gate_bias = self.gates.bias.float().contiguous()            # added to the logits in 32 bits
+        self.scales = [get(n).float().contiguous() for n in self.scale_names]
+
+    def input_norms(self):
+        return [self.norm.as_grouped()]
+
+    def __call__(self, x, ctx, cache, write_cache=True):
+        k = ctx.kernels
+        dtype = ctx.extras.get("activation_dtype", x.dtype)
+        if x.dtype != torch.float32:
+            x = x.float()
+        kept = ctx.extras.pop(self.KEY, None)
+        h = kept[1] if kept is not None and kept[0] is x else k.grouped_rmsnorm(x, *self.norm.as_grouped(), out_dtype=dtype)
+        results = [self.mixer(h, ctx, cache, residual=None, write_cache=write_cache, out_dtype=torch.float32)]
+        if self.feed_forward is not None:
+            results.append(self.feed_forward(h, ctx, residual=None, out_dtype=torch.float32))
+        gates = self.gates(h, ctx, with_bias=False)
+        following = ctx.following_norms
+        if following is not None and (len(following) != 1 or len(following[0]) != 3):                     # (not a norm this kernel forms)
+            following = None
+        x, h = k.gated_combine(x, results, self.scales, gates, self.gate_bias, following[0] if following else None, dtype)
+        if following:
+            ctx.extras[self.KEY] = (x, h)
+        return x
+
+
+BLOCKS.register("shared_norm_gated_residual", SharedNormGatedResidualBlock)

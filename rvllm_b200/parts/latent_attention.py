@@ -19,6 +19,10 @@ head's query becomes [Wuk_h^T q_h | rot(q_h rotated part)] of that width, the at
 leading kv_rank elements as the value, and Wuv_h is applied once per query to the kv_rank-wide result.  A step costs
 the same whatever part of the context it attends to, and nothing per head is ever stored.
 
+With `q_rank` the queries have a low-rank row of their own: cq = rms(Wdq h) * wd (q_rank values), q = Wuq cq.  Then the stacked
+product gives [cq' | c' r | gate logits], one kernel norms both rows, writes the cache and applies the sigmoid, and the
+splitting of q comes after its own product (tensors dq, dq.norm, uq instead of q).
+
 One stacked product gives [q | c' r | gate logits] in float32; one kernel normalises c', rotates, writes the cache row,
 splits q and applies the sigmoid; two products per head (batched over the heads) absorb Wuk into the query and apply
 Wuv to the result.  Sizes and constants are parameters; tensor names default to q, dkv, dkv.norm, uk, uv, g, o.
@@ -36,11 +40,13 @@ from .linear import Linear
 class LatentAttention(Part):
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, value_dim: int, kv_rank: int,
                  scale: float, eps: float, gate: bool = True, position=None, suffix: str = "", sink: bool = False,
-                 pairs: str = "neighbours"):
+                 pairs: str = "neighbours", q_rank: Optional[int] = None):
         from ..errors import ConfigError
         problems = []
         if min(num_heads, head_dim, value_dim, kv_rank) < 1 or rot_dim < 0:
             problems.append("sizes must be positive")
+        if q_rank is not None and q_rank < 1:
+            problems.append(f"the queries' latent needs at least one element, got {q_rank}")
         if rot_dim % 2:
             problems.append(f"the rotated part must have an even size, got {rot_dim}")
         if pairs not in ("neighbours", "halves"):
@@ -54,7 +60,12 @@ class LatentAttention(Part):
         self.position, self.has_sink, self.pairs = position, sink, pairs
         self.q_head = head_dim + rot_dim                 # a head's slice of the query product
         self.row = kv_rank + rot_dim                     # a cached row, and a head's absorbed query
+        self.q_rank = q_rank
         outs, names = [num_heads * self.q_head, self.row], ["q", "dkv"]
+        self.uq = self.q_norm = None
+        if q_rank is not None:
+            outs[0], names[0] = q_rank, "dq"
+            self.uq = Linear(q_rank, [num_heads * self.q_head], ["uq"], suffix=suffix)
         if gate:
             outs.append(num_heads)
             names.append("g")
@@ -64,6 +75,9 @@ class LatentAttention(Part):
 
     def tensor_specs(self):
         sink = {"sink": TensorSpec((self.num_heads,), "bias")} if self.has_sink else {}
+        if self.uq is not None:
+            sink.update(self.uq.tensor_specs())
+            sink["dq.norm"] = TensorSpec((self.q_rank,), "norm")
         return {**self.qdg.tensor_specs(), **self.out.tensor_specs(), **sink,
                 "dkv.norm": TensorSpec((self.kv_rank,), "norm"),
                 "uk": TensorSpec((self.num_heads * self.head_dim, self.kv_rank), "matrix"),
@@ -73,6 +87,9 @@ class LatentAttention(Part):
         self.qdg.bind(get)
         self.out.bind(get)
         self.c_norm = get("dkv.norm")
+        if self.uq is not None:
+            self.uq.bind(get)
+            self.q_norm = get("dq.norm")
         self.sink = get("sink").float().contiguous() if self.has_sink else None        # the softmax is float32
         # per head: Wuk_h^T [kv_rank, dim] (the weight of q_h -> its absorbed part) and Wuv_h [vdim, kv_rank] as stored
         self.uk_t = get("uk").view(self.num_heads, self.head_dim, self.kv_rank).transpose(1, 2).contiguous()
@@ -88,9 +105,17 @@ class LatentAttention(Part):
         cos, sin = tables if tables is not None else (None, None)
         H, R = self.num_heads, self.kv_rank
         proj = self.qdg(x, ctx, out_dtype=torch.float32)          # rounded once, after the norm and the rotation
-        q_plain, q_row, gate = k.latent_prepare(proj, self.c_norm, self.eps, ctx.positions, cos, sin, meta.slot_mapping,
-                                                cache.kv, H, self.head_dim, self.rot_dim, R, x.dtype,
-                                                with_gate=self.has_gate, write_kv=write_cache, halves=self.pairs == "halves")
+        if self.uq is not None:
+            low, gate = k.latent_down(proj, self.q_norm, self.c_norm, self.eps, ctx.positions, cos, sin, meta.slot_mapping, cache.kv,
+                                      self.q_rank, self.rot_dim, R, x.dtype, heads=H if self.has_gate else 0, write_kv=write_cache,
+                                      halves=self.pairs == "halves")
+            q = self.uq(low, ctx, out_dtype=torch.float32)
+            q_plain, q_row = k.latent_queries(q, ctx.positions, cos, sin, H, self.head_dim, self.rot_dim, R, x.dtype,
+                                              halves=self.pairs == "halves")
+        else:
+            q_plain, q_row, gate = k.latent_prepare(proj, self.c_norm, self.eps, ctx.positions, cos, sin, meta.slot_mapping,
+                                                    cache.kv, H, self.head_dim, self.rot_dim, R, x.dtype,
+                                                    with_gate=self.has_gate, write_kv=write_cache, halves=self.pairs == "halves")
         k.head_linear(q_plain, self.uk_t, q_row[:, :, :R])        # the absorbed part of every head's query
         o = k.latent_attention(q_row, cache.kv, meta, H, self.row, R, self.scale, gate=gate, sinks=self.sink)     # [T, H, kv_rank]
         o = k.head_linear(o, self.uv, None)                        # [T, H, vdim]

@@ -14,8 +14,11 @@ choice is a table lookup by token id.
                  s = sigmoid(Wr x) in float32; the choice is made among s + correction (a number per expert), only within
                  the `keep_groups` best of `groups` equal groups of neighbouring experts (a group counts by the sum of its
                  two largest corrected scores); the weights are the chosen experts' s divided by their sum (+ 1e-20).
-                 Optionally a shared expert of the same form runs for every token and is added times
-                 sigmoid(w_sg . x), one number per token.
+                 Scoring "softmax_all": s = softmax(Wr x) over all experts; otherwise as "sigmoid".  A group may count by its
+                 largest corrected score alone (`group_score="max"`).  The last `identity` outputs of the router are experts
+                 without tensors that return x itself.
+                 Optionally a shared expert of the same form runs for every token and is added, by default times
+                 sigmoid(w_sg . x), one number per token (`shared_gate=None`: as it is).
 """
 from __future__ import annotations
 
@@ -99,23 +102,29 @@ class TableMoE(Part):
 
 class RoutedMoE(Part):
     ACTIVATIONS = ("relu2", "silu")
-    SCORINGS = ("sigmoid", "softmax")
+    SCORINGS = ("sigmoid", "softmax", "softmax_all")
+    GROUP_SCORES = ("top2", "max")
 
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, groups: int = 1, keep_groups: int = 1,
                  shared_intermediate_size: Optional[int] = None, activation: str = "relu2", names=None,
                  router: str = "router", correction: str = "correction", expert_prefix: str = "e",
-                 shared_prefix: str = "shared.", shared_gate: str = "sg", suffix: str = "", weight_eps: float = 1e-20,
-                 scoring: str = "sigmoid"):
+                 shared_prefix: str = "shared.", shared_gate: Optional[str] = "sg", suffix: str = "", weight_eps: float = 1e-20,
+                 scoring: str = "sigmoid", identity: int = 0, group_score: str = "top2"):
         from ..errors import ConfigError
         problems = []
-        if not 1 <= top <= experts:
-            problems.append(f"a token uses {top} of {experts} experts")
-        if groups < 1 or experts % max(groups, 1) or not 1 <= keep_groups <= groups:
-            problems.append(f"{experts} experts in {groups} equal groups of which {keep_groups} are kept")
-        elif top > keep_groups * (experts // groups):
-            problems.append(f"{top} experts per token out of {keep_groups} groups of {experts // groups}")
-        if experts > 1024:
-            problems.append(f"the router serves at most 1,024 experts, got {experts}")
+        outputs = experts + identity                         # of the router
+        if experts < 1 or identity < 0:
+            problems.append(f"{experts} experts and {identity} identity experts")
+        if not 1 <= top <= outputs:
+            problems.append(f"a token uses {top} of {outputs} experts")
+        if groups < 1 or outputs % max(groups, 1) or not 1 <= keep_groups <= groups:
+            problems.append(f"{outputs} experts in {groups} equal groups of which {keep_groups} are kept")
+        elif top > keep_groups * (outputs // groups):
+            problems.append(f"{top} experts per token out of {keep_groups} groups of {outputs // groups}")
+        if outputs > 1024:
+            problems.append(f"the router serves at most 1,024 experts, got {outputs}")
+        if group_score not in self.GROUP_SCORES:
+            problems.append(f"group score {group_score!r} is not known ({', '.join(self.GROUP_SCORES)})")
         if activation not in self.ACTIVATIONS:
             problems.append(f"expert activation {activation!r} is not known ({', '.join(self.ACTIVATIONS)})")
         if scoring not in self.SCORINGS:
@@ -124,7 +133,8 @@ class RoutedMoE(Part):
             raise ConfigError(problems, "routed mixture of experts")
         self.hidden_size, self.intermediate_size, self.experts, self.top = hidden_size, intermediate_size, experts, top
         self.groups, self.keep_groups, self.activation, self.weight_eps = groups, keep_groups, activation, weight_eps
-        self.scoring, self.gated = scoring, activation == "silu"
+        self.scoring, self.gated, self.identity, self.group_score = scoring, activation == "silu", identity, group_score
+        self.outputs = outputs
         names = tuple(names) if names is not None else (("gate", "up", "down") if self.gated else ("up", "down"))
         self.names, self.router_name, self.correction_name, self.expert_prefix = names, router, correction, expert_prefix
         self.shared_prefix, self.shared_gate, self.suffix = shared_prefix, shared_gate, suffix
@@ -142,8 +152,8 @@ class RoutedMoE(Part):
 
     def tensor_specs(self):
         *first, d = self.names                               # (gate and) up, down
-        specs = {self.router_name + self.suffix: TensorSpec((self.experts, self.hidden_size), "matrix"),
-                 self.correction_name: TensorSpec((self.experts,), "bias")}
+        specs = {self.router_name + self.suffix: TensorSpec((self.outputs, self.hidden_size), "matrix"),
+                 self.correction_name: TensorSpec((self.outputs,), "bias")}
         for e in range(self.experts):
             p = f"{self.expert_prefix}{e}."
             for u in first:
@@ -152,14 +162,16 @@ class RoutedMoE(Part):
         if self.shared_ff is not None:
             for part in self._shared_parts():
                 specs.update({self.shared_prefix + n: ts for n, ts in part.tensor_specs().items()})
-            specs[self.shared_prefix + self.shared_gate + self.suffix] = TensorSpec((1, self.hidden_size), "matrix")
+            if self.shared_gate is not None:
+                specs[self.shared_prefix + self.shared_gate + self.suffix] = TensorSpec((1, self.hidden_size), "matrix")
         return specs
 
     def bind(self, get):
         *first, d = self.names
         rows = [get(self.router_name + self.suffix)]
-        if self.shared_ff is not None:                       # the shared expert's gate is one more row of the router's product
-            rows.append(get(self.shared_prefix + self.shared_gate + self.suffix))
+        if self.shared_ff is not None:
+            if self.shared_gate is not None:                 # the shared expert's gate is one more row of the router's product
+                rows.append(get(self.shared_prefix + self.shared_gate + self.suffix))
             for part in self._shared_parts():
                 part.bind(lambda name: get(self.shared_prefix + name))
         self.router = torch.cat(rows, dim=0).contiguous()
@@ -172,25 +184,29 @@ class RoutedMoE(Part):
     def __call__(self, x, ctx, residual=None, out_dtype=None):
         k = ctx.kernels
         scores = k.linear(x, self.router, None, None, torch.float32)
-        chosen, weights, shared_gate = k.moe_route_top(scores, self.correction, self.experts, self.top, self.groups,
-                                                       self.keep_groups, self.weight_eps, shared_gate=self.shared_ff is not None,
-                                                       scoring=self.scoring)
+        options = {} if self.group_score == "top2" else {"group_score": self.group_score}
+        with_gate = self.shared_ff is not None and self.shared_gate is not None
+        chosen, weights, shared_gate = k.moe_route_top(scores, self.correction, self.outputs, self.top, self.groups,
+                                                       self.keep_groups, self.weight_eps, shared_gate=with_gate,
+                                                       scoring=self.scoring, **options)
+        given = {"weights": weights, "activation": self.activation}
+        if self.identity:                                    # numbers beyond the experts name the identity
+            given["identity"] = True
         if self.shared is not None and residual is None:     # the shared expert's gate is a factor on what the experts' sum adds
             add = self.shared(x, ctx, out_dtype=torch.float32)
-            return k.moe_experts(x, chosen, self.up, self.down, 1.0, add=add, out_dtype=out_dtype or x.dtype, weights=weights,
-                                 activation=self.activation, add_scale=shared_gate)
+            return k.moe_experts(x, chosen, self.up, self.down, 1.0, add=add, out_dtype=out_dtype or x.dtype,
+                                 add_scale=shared_gate, **given)
         add = residual
         if self.shared is not None:
             add = k.moe_experts(x, chosen, self.up, self.down, 1.0, add=self.shared(x, ctx, out_dtype=torch.float32),
-                                out_dtype=torch.float32, weights=weights, activation=self.activation, add_scale=shared_gate)
+                                out_dtype=torch.float32, add_scale=shared_gate, **given)
             add = k.scaled_sum(add, 1.0, residual if residual.dtype == torch.float32 else residual.float(), 1.0)
             return add if out_dtype == torch.float32 else add.to(out_dtype or x.dtype)
         if self.shared_up is not None:
             u = self.shared_up(x, ctx, out_dtype=torch.float32)
             a = k.act_rows(u, self.activation, x.dtype, row_scale=shared_gate)      # W (g a) = g (W a): the gate rides on the activation
             add = self.shared_down(a, ctx, residual=residual, out_dtype=torch.float32)
-        return k.moe_experts(x, chosen, self.up, self.down, 1.0, add=add, out_dtype=out_dtype or x.dtype, weights=weights,
-                             activation=self.activation)
+        return k.moe_experts(x, chosen, self.up, self.down, 1.0, add=add, out_dtype=out_dtype or x.dtype, **given)
 
 
 FEED_FORWARDS.register("polynorm_mlp", PolyNormMLP)

@@ -40,6 +40,34 @@ class RMSNorm(Part):
 NORMS.register("rmsnorm", RMSNorm)
 
 
+class GroupedRMSNorm(Part):
+    """The row in `groups` equal consecutive parts, each over its own root mean square: y = x / sqrt(mean(part^2) + eps) * gamma.
+    Arithmetic in float32; the result has the activations' type."""
+
+    def __init__(self, size: int, groups: int, eps: float, tensor: str = "weight"):
+        from ..errors import ConfigError
+        if groups < 1 or size % groups:
+            raise ConfigError(f"a norm over rows of {size} cannot have {groups} equal groups")
+        self.size, self.groups, self.eps, self.tensor = size, groups, eps, tensor
+        self.weight = None
+
+    def tensor_specs(self):
+        return {self.tensor: TensorSpec((self.size,), "norm")}
+
+    def bind(self, get):
+        self.weight = get(self.tensor)
+
+    def __call__(self, x, ctx):
+        return ctx.kernels.grouped_rmsnorm(x, *self.as_grouped(), out_dtype=ctx.extras.get("activation_dtype", x.dtype))
+
+    def as_grouped(self):
+        """(gamma, eps, groups) for a block that applies this norm inside a fused kernel."""
+        return self.weight, self.eps, self.groups
+
+
+NORMS.register("grouped_rmsnorm", GroupedRMSNorm)
+
+
 class DynamicTanh(Part):
     """y = tanh(alpha x) * weight + bias, element by element: a norm that forms no statistic of the row.  `alpha` is one
     number, stored beside the weight as `<tensor>.alpha`; the bias as `<tensor>.b`.  Arithmetic in float32; the three

@@ -13,7 +13,7 @@ float tensor becomes float32.
 from __future__ import annotations
 
 import fnmatch
-from typing import Dict, Iterable, Tuple
+from typing import Dict, Iterable, Optional, Tuple
 
 import torch
 
@@ -42,13 +42,20 @@ class WeightSource:
         self.model_dir = model_dir
         self.entries: Dict[str, TensorEntry] = open_model_files(model_dir)
 
-    def check(self, expected: Dict[str, Tuple[int, ...]], ignored: Iterable[str] = ()) -> None:
+    def check(self, expected: Dict[str, Tuple[int, ...]], ignored: Iterable[str] = (), free: Optional[Dict[str, Tuple[int, ...]]] = None) -> None:
+        """`free`: per tensor, the dimensions whose size is the file's own (at least 1)."""
         ignored = tuple(ignored)
+        free = free or {}
+
+        def fits(name: str) -> bool:
+            have, want, open_dims = tuple(self.entries[name].shape), tuple(expected[name]), free.get(name, ())
+            return len(have) == len(want) and all(h == w or (i in open_dims and h > 0) for i, (h, w) in enumerate(zip(have, want)))
+
         missing = [n for n in expected if n not in self.entries]
         unexpected = [n for n in self.entries if n not in expected
                       and not any(fnmatch.fnmatch(n, pat) for pat in ignored)]
         wrong = [f"{n}: expected {list(expected[n])}, file has {list(self.entries[n].shape)}"
-                 for n in expected if n in self.entries and tuple(self.entries[n].shape) != tuple(expected[n])]
+                 for n in expected if n in self.entries and not fits(n)]
         if missing or unexpected or wrong:
             raise LoaderError("checkpoint tensors do not match the model", path=self.model_dir,
                               missing=sorted(missing), unexpected=sorted(unexpected), wrong_shape=sorted(wrong))

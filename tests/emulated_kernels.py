@@ -91,6 +91,19 @@ class EmulatedKernels:
         gate = torch.sigmoid(x[:, qw + row:qw + row + num_heads]) if with_gate else None
         return q_plain, q_row, gate
 
+    def latent_down(self, proj, q_gamma, c_gamma, eps, positions, cos, sin, slot_mapping, cache_layer, q_rank, rot_dim, kv_rank,
+                    out_dtype, heads=0, write_kv=True, halves=False):
+        rest = torch.cat([torch.zeros((proj.shape[0], 1 + rot_dim)), proj[:, q_rank:q_rank + kv_rank + rot_dim].float()], dim=1)
+        self.latent_prepare(rest, c_gamma, eps, positions, cos, sin, slot_mapping, cache_layer, 1, 1, rot_dim, kv_rank, out_dtype,
+                            with_gate=False, write_kv=write_kv, halves=halves)
+        gate = torch.sigmoid(proj[:, q_rank + kv_rank + rot_dim:].float()) if heads else None
+        return self.rmsnorm(proj[:, :q_rank].float(), q_gamma, eps).to(out_dtype), gate
+
+    def latent_queries(self, q, positions, cos, sin, num_heads, head_dim, rot_dim, kv_rank, out_dtype, halves=False):
+        full = torch.cat([q.float(), torch.zeros((q.shape[0], kv_rank + rot_dim))], dim=1)
+        return self.latent_prepare(full, torch.ones(kv_rank), 1.0, positions, cos, sin, None, None, num_heads, head_dim, rot_dim, kv_rank,
+                                   out_dtype, with_gate=False, write_kv=False, halves=halves)[:2]
+
     def head_linear(self, x, weight, out=None, out_dtype=None):
         y = torch.einsum("thk,hnk->thn", x.float(), weight.float()).contiguous()
         if out is None:
@@ -126,13 +139,17 @@ class EmulatedKernels:
         return out
 
     def moe_experts(self, x, chosen, gate_up, down, weight, add=None, out_dtype=None, weights=None, activation="silu",
-                    add_scale=None):
+                    add_scale=None, identity=False):
         T, ff = x.shape[0], gate_up.shape[1] // 2
         out = torch.zeros((T, x.shape[1])) if add is None else add.clone().float()
         if add_scale is not None:
             out *= add_scale[:, None]
         for t in range(T):
             for j, e in enumerate(chosen[t].tolist()):
+                if e >= gate_up.shape[0]:         # an expert without matrices
+                    if identity:
+                        out[t] += weight * (float(weights[t, j]) if weights is not None else 1.0) * x[t].float()
+                    continue
                 gu = gate_up[e].float() @ x[t].float()
                 if activation == "relu2":         # plain experts: every row of the first matrix is an up row
                     a = torch.relu(gu) ** 2
@@ -161,21 +178,23 @@ class EmulatedKernels:
             a = a * row_scale[:, None]
         return a.to(out_dtype)
 
-    def moe_route_top(self, scores, correction, experts, top, groups, keep, weight_eps, shared_gate=False, scoring="sigmoid"):
-        s = torch.sigmoid(scores[:, :experts].float()) if scoring == "sigmoid" else scores[:, :experts].float()
+    def moe_route_top(self, scores, correction, experts, top, groups, keep, weight_eps, shared_gate=False, scoring="sigmoid",
+                      group_score="top2"):
+        s = {"sigmoid": torch.sigmoid, "softmax": lambda z: z, "softmax_all": lambda z: torch.softmax(z, -1)}[scoring](scores[:, :experts].float())
         c = s + correction
         per = experts // groups
-        gs = c.view(-1, groups, per).topk(min(2, per), dim=-1).values.sum(-1)
+        gs = c.view(-1, groups, per).topk(min(2 if group_score == "top2" else 1, per), dim=-1).values.sum(-1)
         kept = gs.topk(keep, dim=-1).indices
         allowed = torch.zeros_like(gs, dtype=torch.bool).scatter_(1, kept, True).repeat_interleave(per, dim=1)
         chosen = c.masked_fill(~allowed, float("-inf")).topk(top, dim=-1).indices
-        w = s.gather(1, chosen) if scoring == "sigmoid" else torch.softmax(c.gather(1, chosen), -1)
+        w = s.gather(1, chosen) if scoring != "softmax" else torch.softmax(c.gather(1, chosen), -1)
         w = w / (w.sum(-1, keepdim=True) + weight_eps)
         gate = torch.sigmoid(scores[:, experts].float()) if shared_gate else None
         return chosen.to(torch.int32), w, gate
 
     def qk_prepare(self, proj, positions, cos, sin, slot_mapping, cache_layer, num_heads, num_kv_heads, head_dim, value_dim,
-                   slot_dim, out_dtype, eps=None, halves=False, with_gate=False, write_kv=True, maps=1, bias=None, value_tables=None):
+                   slot_dim, out_dtype, eps=None, halves=False, with_gate=False, write_kv=True, maps=1, bias=None, value_tables=None,
+                   norms=None, temperature=None, keep_values=None, mix_values=None):
         T = proj.shape[0]
         x = proj.float().clone()
         if bias is not None:
@@ -198,18 +217,30 @@ class EmulatedKernels:
             return out
 
         def norm(v):
-            return v if eps is None else v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)
+            return v if eps is None or norms is not None else v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)
+
+        def weighted(v, which):          # in front of the rotation
+            return v if norms is None else v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * norms[which]
 
         qw = num_heads * maps * head_dim
-        turned = norm(turn(x[:, :qw].view(T, num_heads, maps, head_dim), cos, sin))
+        turned = norm(turn(weighted(x[:, :qw].reshape(T, num_heads, maps, head_dim), 0), cos, sin))
+        if temperature is not None:
+            coef, every = temperature
+            grown = 1.0 + coef * torch.log(torch.div(pos + 1, every, rounding_mode="floor").float() + 1.0)
+            turned = turned * grown.view(T, 1, 1, 1)
         q = torch.zeros((T, num_heads, maps, slot_dim))
         for m in range(maps):
             q[:, :, m, m * head_dim:(m + 1) * head_dim] = turned[:, :, m]
         col = qw
         if write_kv:
             kw, vw = num_kv_heads * maps * head_dim, num_kv_heads * value_dim
-            k = norm(turn(x[:, col:col + kw].view(T, num_kv_heads, maps, head_dim), cos, sin)).reshape(T, num_kv_heads, maps * head_dim)
-            v = x[:, col + kw:col + kw + vw].view(T, num_kv_heads, value_dim)
+            k = norm(turn(weighted(x[:, col:col + kw].reshape(T, num_kv_heads, maps, head_dim), 1), cos, sin)).reshape(T, num_kv_heads, maps * head_dim)
+            v = x[:, col + kw:col + kw + vw]
+            if keep_values is not None:
+                keep_values.copy_(v)
+            if mix_values is not None:
+                v = (1.0 - mix_values[1]) * v + mix_values[1] * mix_values[0]
+            v = v.reshape(T, num_kv_heads, value_dim)
             if value_tables is not None:
                 v = turn(v, *value_tables)
             col += kw + vw
@@ -240,6 +271,11 @@ class EmulatedKernels:
         out[..., first], out[..., second] = a * c + b * s, b * c - a * s
         return out.reshape(T, heads * value_dim).to(o.dtype)
 
+    def gate_elements(self, o, proj, col0, heads, value_dim, slot_dim):
+        T = o.shape[0]
+        g = torch.sigmoid(proj[:, col0:col0 + heads * value_dim].float())
+        return (o.view(T, heads, slot_dim)[..., :value_dim].reshape(T, -1).float() * g).to(o.dtype)
+
     def map_difference(self, o, lam, eps, factor, heads, value_dim, slot_dim):
         T = o.shape[0]
         v = o.view(T, heads, 2, slot_dim)[..., :value_dim].float()
@@ -251,6 +287,18 @@ class EmulatedKernels:
         for y, c in terms:
             x += c * y
         return x, [self.rmsnorm(x, gamma, eps).to(out_dtype) for gamma, eps in norms]
+
+    def grouped_rmsnorm(self, x, gamma, eps, groups, out_dtype=None):
+        parts = x.float().view(x.shape[0], groups, -1)
+        y = parts / torch.sqrt((parts * parts).mean(-1, keepdim=True) + eps)
+        return (y.reshape(x.shape) * gamma.float()).to(out_dtype or x.dtype)
+
+    def gated_combine(self, x, terms, scales, gates, bias, norm, out_dtype):
+        cols = x.shape[1]
+        for i, (y, s) in enumerate(zip(terms, scales)):
+            span = slice(i * cols, (i + 1) * cols)
+            x += y * s * torch.sigmoid(gates[:, span].float() + bias[span])
+        return x, (self.grouped_rmsnorm(x, *norm, out_dtype=out_dtype) if norm is not None else None)
 
     def mingru(self, proj, z_bias, x_bias, cu_seqlens, state_slots, state, width, single, out_dtype):
         out = torch.zeros((proj.shape[0], width))
@@ -444,7 +492,7 @@ class EmulatedKernels:
                                      num_heads, num_kv_heads, head_dim)
 
     def paged_attention(self, q, cache_layer, meta, num_heads, num_kv_heads, head_dim, scale, window,
-                        softcap=None, sinks=None, gate=None):
+                        softcap=None, sinks=None, gate=None, distance_bias=None):
         T = q.shape[0]
         ps = cache_layer.shape[3]
         out = torch.zeros_like(q).view(T, num_heads, head_dim)
@@ -471,6 +519,9 @@ class EmulatedKernels:
                     sc = (K @ qv[t, h]) * scale
                     if softcap is not None:
                         sc = softcap * torch.tanh(sc / softcap)
+                    if distance_bias is not None:
+                        by_distance = distance_bias.natural[g, :, h - g * (num_heads // num_kv_heads)]
+                        sc = sc + by_distance[(pos - torch.tensor(keys)).clamp(max=len(by_distance) - 1)]
                     if sinks is not None:
                         p = torch.softmax(torch.cat([sc, sinks[h:h + 1].float()]), 0)[:-1]
                     else:
