@@ -78,6 +78,8 @@ class _Reader(NumberReader):
             out["bias_rows"] = self.integer(m, "bias_rows", at, minimum=2) if "bias_rows" in m else DEFAULT_BIAS_ROWS
             temp = m.get("q_temp")
             out["temp_coef"] = None if temp is None else self.number(temp, "coef", at + "q_temp: ", positive=False)
+            if isinstance(temp, dict) and isinstance(temp.get("every"), float) and temp["every"].is_integer():
+                temp = dict(temp, every=int(temp["every"]))
             out["temp_every"] = None if temp is None else self.integer(temp, "every", at + "q_temp: ")
         else:
             out["rot_dims"], out["rot_base"] = self.rotation(m, at, out["dim"], "dim")
