@@ -2,7 +2,7 @@
 """Benchmark of the engine on one B200: decode tokens per second, prefill, roofline.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers L] [--shape NAME]
-                    [--workload decode|serve|tufirax|vipelix|tibepel|tugodra|sozudra] [--impl ours|reference]
+                    [--workload decode|serve|tufirax|vipelix|tibepel|tugodra|sozudra|lefolorn] [--impl ours|reference]
 
 The default run has the layer sizes of Llama-3.1-8B (32 layers, hidden 4096, 32 query heads,
 8 key/value heads of 128, MLP 14336, vocabulary 128256, llama3 rotary scaling) with random
@@ -1272,6 +1272,184 @@ def run_sozudra(args):
 
 
 # ---------------------------------------------------------------------------------------------------------
+# --workload lefolorn: the Lefolorn design (one norm in groups in front of a mixer and routed experts that stand side by side,
+# both scaled and gated element by element; window attention on normed queries and keys, latent attention with low-rank
+# queries and a sink, attention with a bias per distance and an element-wise gate; a softmax router with identity experts) at
+# layer sizes that resemble real models, beside the Tugodra decoder of this engine - the closest design: window attention on
+# unit-norm queries and keys, latent attention with a sink, routed experts with a shared one, a float32 stream - at the same
+# width, depth, heads, window, latent and experts; then each of the design's own kernels alone beside the like kernel of the
+# engine's other designs, with its bytes or FLOPs over its time against the measured copy bandwidth or bf16 peak.  Random
+# weights; its own JSON line.
+LEFOLORN_SIZES = {
+    "2k": dict(width=2048, heads=16, kv=4, dim=128, window=1024, l_dim=128, rot=64, rank=192, q_rank=768, groups=4, e_ff=1408, experts=14,
+               identity=2, top=2, e_groups=4, keep=2, shared=2816, bias_max=512, layers=8),
+    "4k": dict(width=4096, heads=32, kv=8, dim=128, window=1024, l_dim=128, rot=64, rank=192, q_rank=1536, groups=4, e_ff=2048, experts=28,
+               identity=4, top=4, e_groups=8, keep=4, shared=4096, bias_max=1024, layers=8),
+}
+
+
+def lefolorn_pair(size: dict, vocab: int = 32768):
+    """(Lefolorn configuration, Tugodra configuration): layers of window attention, latent attention, attention with a distance
+    bias and latent attention, in turn, each with experts; beside as many Tugodra layers of window and latent attention in turn."""
+    E = size["experts"] + size["identity"]
+    groups = {"count": size["e_groups"], "keep": size["keep"]}
+    mlp = {"kind": "moe", "expert": {"ff": size["e_ff"]}, "shared": {"ff": size["shared"]},
+           "router": {"experts": size["experts"], "identity": size["identity"], "top": size["top"], "groups": groups}}
+    heads = {"heads": size["heads"], "kv_heads": size["kv"], "dim": size["dim"], "vdim": size["dim"], "scale": size["dim"] ** -0.5}
+    lat = {"heads": size["heads"], "dim": size["l_dim"], "rot_dim": size["rot"], "vdim": size["l_dim"], "kv_rank": size["rank"],
+           "scale": (size["l_dim"] + size["rot"]) ** -0.5, "rot": {"dims": size["rot"], "base": 500000.0}}
+    win = {"type": "attention_2", "mlp": mlp, "mixer": dict(heads, softcap=30.0, mask={"size": size["window"]}, v_mix=True,
+                                                            rot={"dims": size["dim"], "base": 1e6})}
+    rel = {"type": "attention", "mlp": mlp, "mixer": dict(heads, bias_max=size["bias_max"], q_temp={"coef": 0.1, "every": 512}, v_mix=True)}
+    low = {"type": "latent_attention", "mlp": mlp, "mixer": dict(lat, q_rank=size["q_rank"])}
+    lef = {"architecture": "Lefolorn", "width": size["width"], "vocab": vocab, "norm": {"eps": 1e-6, "groups": size["groups"]},
+           "layers": [win, low, rel, low] * (size["layers"] // 4)}
+    t_mlp = dict(mlp, router={"experts": E, "top": size["top"], "groups": groups})
+    t_att = {"type": "attention", "mlp": t_mlp, "mixer": dict(heads, mask={"size": size["window"]}, rot={"dims": size["dim"], "base": 1e6})}
+    tug = {"architecture": "Tugodra", "width": size["width"], "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": size["width"] ** 0.5},
+           "layers": [t_att, {"type": "latent_attention", "mlp": t_mlp, "mixer": lat}] * (size["layers"] // 2)}
+    return lef, tug
+
+
+def run_lefolorn(args):
+    import torch
+
+    from rvllm_b200.kernels import AttentionMeta
+    from rvllm_b200.parts.distance import distance_table
+
+    peaks = measured_peaks()
+    PROMPT, CTX, batch = 2048, 4096, args.batch
+    gen = torch.Generator().manual_seed(0)
+    out = {"workload": "lefolorn", "dtype": "bf16", "data": "synthetic", "peaks": peaks["source"], "prompt_len": PROMPT, "batch": batch,
+           "steps": args.steps, "warmup": args.warmup, "models": {}, "kernels": {}}
+    K = None
+    for name in (args.sizes.split(",") if args.sizes else list(LEFOLORN_SIZES)):
+        lef, tug = lefolorn_pair(LEFOLORN_SIZES[name])
+        a, K = measure_design(lef, args, gen, PROMPT, CTX)
+        b, K = measure_design(tug, args, gen, PROMPT, CTX)
+        out["models"][name] = {"lefolorn": a, "tugodra_same_size": b, "layers": LEFOLORN_SIZES[name]["layers"],
+                               "prefill_ratio": round(a["prefill_tok_s"] / b["prefill_tok_s"], 3),
+                               "decode_ratio": round(a["decode_tok_s"] / b["decode_tok_s"], 3)}
+
+    # ---- the design's kernels alone, at the "4k" sizes, beside the like kernel ---------------------------------------
+    torch.manual_seed(0)
+    z = LEFOLORN_SIZES["4k"]
+    dev, bf = "cuda", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    bw, peak = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    timed = lambda fn: _time_kernel(fn, flush=flush)
+
+    def by_bytes(name, fn, nbytes, like_name, like_fn, like_bytes):
+        ms_like, ms = timed(like_fn), timed(fn)
+        frac, lfrac = nbytes / (ms / 1e3) / bw, like_bytes / (ms_like / 1e3) / bw
+        out["kernels"][name] = {"ms": round(ms, 4), "gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(frac, 4), "farther_than_like": round(lfrac / frac, 2),
+                                "like": {"kernel": like_name, "ms": round(ms_like, 4), "frac_hbm": round(lfrac, 4)}}
+
+    def by_flops(name, fn, flops, like_name, like_fn, like_flops):
+        ms_like, ms = timed(like_fn), timed(fn)
+        frac, lfrac = flops / (ms / 1e3) / peak, like_flops / (ms_like / 1e3) / peak
+        out["kernels"][name] = {"ms": round(ms, 4), "tflops": round(flops / ms / 1e9, 1), "frac_bf16": round(frac, 4), "farther_than_like": round(lfrac / frac, 2),
+                                "like": {"kernel": like_name, "ms": round(ms_like, 4), "frac_bf16": round(lfrac, 4)}}
+
+    W, H, G, D, WIN = z["width"], z["heads"], z["kv"], z["dim"], z["window"]
+    LD, RD, R, RQ = z["l_dim"], z["rot"], z["rank"], z["q_rank"]
+    ROW, pages = R + RD, PROMPT // 16
+    pos = torch.arange(PROMPT, dtype=torch.int32, device=dev)
+
+    def tables(dims):
+        ang = torch.arange(PROMPT, dtype=torch.float64)[:, None] * torch.tensor([1e6 ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)[None, :]
+        return torch.cos(ang).float().to(dev), torch.sin(ang).float().to(dev)
+
+    cos, sin = tables(D)
+    cos_l, sin_l = tables(RD)
+    g = torch.ones(W, dtype=bf, device=dev)
+    cache = torch.zeros(pages, 2, G, 16, D, dtype=bf, device=dev)
+    cache1 = torch.zeros(pages, 1, 1, 16, ROW, dtype=bf, device=dev)
+    for label, T in (("prefill", PROMPT), ("decode", batch)):
+        # -- the stream, its gates and the norm of the next layer
+        x, y1, y2 = (torch.randn(T, W, device=dev) for _ in range(3))
+        gates, gb, s1 = torch.randn(T, 2 * W, device=dev).to(bf), torch.zeros(2 * W, device=dev), torch.ones(W, device=dev)
+        by_bytes(f"gated_combine_{label}", lambda: K.gated_combine(x, [y1, y2], [s1, s1], gates, gb, (g, 1e-6, z["groups"]), bf), T * W * (8 + 8 + 4 + 2),
+                 "stream_combine, two terms and a norm", lambda: K.stream_combine(x, [(y1, 0.4), (y2, 0.8)], [(g, 1e-6)], bf), T * W * 18)
+        by_bytes(f"grouped_rmsnorm_{label}", lambda: K.grouped_rmsnorm(x, g, 1e-6, z["groups"], out_dtype=bf), T * W * 6,
+                 "rmsnorm", lambda: K.rmsnorm(x, g, 1e-6, out_dtype=bf), T * W * 6)
+
+        # -- around the attention kernels
+        p_ = pos[:T].contiguous()
+        cols = (H + 2 * G) * D
+        pr_like, pr = torch.randn(T, cols + H, device=dev), torch.randn(T, cols, device=dev)
+        prg = torch.randn(T, cols + H * D, device=dev)
+        bias, gam, first = torch.randn(cols, device=dev), torch.ones(D, device=dev), torch.randn(T, G * D, device=dev)
+        like = ("qk_unit_prepare with a gate", lambda: K.qk_unit_prepare(pr_like, 1e-6, p_, cos, sin, p_, cache, H, G, D, D, D, bf),
+                T * (pr_like.shape[1] * 4 + cols * 2 + H * 4))
+        by_bytes(f"qk_prepare_norms_rotation_{label}", lambda: K.qk_prepare(pr, p_, cos, sin, p_, cache, H, G, D, D, D, bf, eps=1e-6, bias=bias, norms=(gam, gam),
+                                                                          mix_values=(first, 0.3)), T * (cols * 6 + G * D * 4), *like)
+        by_bytes(f"qk_prepare_norms_temperature_{label}", lambda: K.qk_prepare(prg[:, :cols], p_, None, None, p_, cache, H, G, D, D, D, bf, eps=1e-6, bias=bias,
+                                                                             norms=(gam, gam), temperature=(0.1, 512), mix_values=(first, 0.3)), T * (cols * 6 + G * D * 4), *like)
+        o1 = torch.randn(T, H * D, device=dev).to(bf)
+        of, gn, zg = torch.randn(T, H * D, device=dev), torch.ones(D, dtype=bf, device=dev), torch.randn(T, H * D, device=dev)
+        by_bytes(f"gate_elements_{label}", lambda: K.gate_elements(o1, prg, cols, H, D, D), T * H * D * 8,
+                 "head_norm_gate", lambda: K.head_norm_gate(of, gn, 1e-6, zg, 0, H, D, bf), T * H * D * 10)
+        pl = torch.randn(T, H * (LD + RD) + ROW, device=dev)
+        pd, ql = torch.randn(T, RQ + ROW, device=dev), torch.randn(T, H * (LD + RD), device=dev)
+        cg, qg = torch.ones(R, dtype=bf, device=dev), torch.ones(RQ, dtype=bf, device=dev)
+        like = ("latent_prepare", lambda: K.latent_prepare(pl, cg, 1e-6, p_, cos_l, sin_l, p_, cache1, H, LD, RD, R, bf, with_gate=False),
+                T * (pl.shape[1] * 4 + (H * (LD + RD) + ROW) * 2))
+        by_bytes(f"latent_down_{label}", lambda: K.latent_down(pd, qg, cg, 1e-6, p_, cos_l, sin_l, p_, cache1, RQ, RD, R, bf), T * (RQ + ROW) * 6, *like)
+        by_bytes(f"latent_queries_{label}", lambda: K.latent_queries(ql, p_, cos_l, sin_l, H, LD, RD, R, bf), T * H * (LD + RD) * 6, *like)
+
+        # -- the router, and gated experts some of whose choices are the identity
+        E, N, top_k, EF = z["experts"], z["experts"] + z["identity"], z["top"], z["e_ff"]
+        corr = torch.zeros(N, device=dev)
+        logits, xb, add = torch.randn(T, N, device=dev), torch.randn(T, W, device=dev).to(bf), torch.randn(T, W, device=dev)
+        n = T * (N * 4 + top_k * 8)
+        by_bytes(f"moe_route_top_softmax_all_{label}", lambda: K.moe_route_top(logits, corr, N, top_k, z["e_groups"], z["keep"], 1e-20, scoring="softmax_all", group_score="max"), n,
+                 "moe_route_top (sigmoid)", lambda: K.moe_route_top(logits, corr, N, top_k, z["e_groups"], z["keep"], 1e-20), n)
+        chosen, wts, _ = K.moe_route_top(logits, corr, N, top_k, z["e_groups"], z["keep"], 1e-20, scoring="softmax_all", group_score="max")
+        real = chosen % E
+        gate_up, down = torch.randn(E, 2 * EF, W, device=dev).to(bf) * 0.02, torch.randn(E, W, EF, device=dev).to(bf) * 0.02
+        mixed = lambda: K.moe_experts(xb, chosen, gate_up, down, 1.0, add=add, out_dtype=torch.float32, weights=wts, identity=True)
+        plain = lambda: K.moe_experts(xb, real, gate_up, down, 1.0, add=add, out_dtype=torch.float32, weights=wts)
+        work = int((chosen < E).sum())
+        if label == "prefill":
+            by_flops("identity_experts_prefill", mixed, 6.0 * work * EF * W, "gated experts, none the identity", plain, 6.0 * T * top_k * EF * W)
+        else:
+            touched, touched_like = len(set(chosen[chosen < E].flatten().tolist())), len(set(real.flatten().tolist()))
+            by_bytes("identity_experts_decode", mixed, touched * 3 * EF * W * 2, "gated experts, none the identity", plain, touched_like * 3 * EF * W * 2)
+        out["kernels"][f"identity_experts_{label}"]["identity_share"] = round(1.0 - work / (T * top_k), 3)
+        del gate_up, down
+
+    # -- attention with a bias per distance and one in the denominator, and window attention with a cap
+    def paged_case(q_len, ctx, seqs):
+        n = seqs * (ctx // 16)
+        kv = torch.randn(n, 2, G, 16, D, device=dev).to(bf)
+        tbl = torch.arange(n, dtype=torch.int32, device=dev).view(seqs, ctx // 16)
+        cu = torch.arange(seqs + 1, dtype=torch.int32, device=dev) * q_len
+        meta = AttentionMeta(tbl, cu, torch.full((seqs,), ctx, dtype=torch.int32, device=dev),
+                             torch.arange(seqs, dtype=torch.int32, device=dev).repeat_interleave(q_len), None, seqs, q_len, ctx, 16,
+                             seqs if q_len == 1 else 0)
+        return torch.randn(seqs * q_len, H * D, device=dev).to(bf), kv, meta, torch.rand(seqs * q_len, H, device=dev)
+
+    dist = distance_table(torch.randn(32, H, device=dev), z["bias_max"], G)
+    one = torch.zeros(H, device=dev)
+    q, kv, meta, gate = paged_case(PROMPT, PROMPT, 1)
+    full = 4.0 * H * D * PROMPT * PROMPT / 2
+    by_flops("distance_bias_attention_prefill", lambda: K.paged_attention(q, kv, meta, H, G, D, 0.09, None, sinks=one, distance_bias=dist), full,
+             "attention with a sink", lambda: K.paged_attention(q, kv, meta, H, G, D, 0.09, None, sinks=one), full)
+    seen = 4.0 * H * D * sum(min(i + 1, WIN) for i in range(PROMPT))
+    by_flops("window_attention_cap_prefill", lambda: K.paged_attention(q, kv, meta, H, G, D, 0.09, WIN, softcap=30.0), seen,
+             "window attention with a gate", lambda: K.paged_attention(q, kv, meta, H, G, D, 0.09, WIN, gate=gate), seen)
+    q2, kv2, meta2, gate2 = paged_case(1, PROMPT, batch)
+    nb = batch * PROMPT * 2 * G * D * 2
+    by_bytes("distance_bias_attention_decode", lambda: K.paged_attention(q2, kv2, meta2, H, G, D, 0.09, None, sinks=one, distance_bias=dist), nb,
+             "attention with a sink", lambda: K.paged_attention(q2, kv2, meta2, H, G, D, 0.09, None, sinks=one), nb)
+    by_bytes("window_attention_cap_decode", lambda: K.paged_attention(q2, kv2, meta2, H, G, D, 0.09, WIN, softcap=30.0), batch * WIN * 2 * G * D * 2,
+             "window attention with a gate", lambda: K.paged_attention(q2, kv2, meta2, H, G, D, 0.09, WIN, gate=gate2), batch * WIN * 2 * G * D * 2)
+    K.raise_on_abort()
+    print(json.dumps(out))
+
+
+# ---------------------------------------------------------------------------------------------------------
 # --workload tibepel: the Tibepel design (chunked attention whose softmax weights are mixed across the heads beside a
 # gated delta rule, mamba1 scans, clamped gated feed-forwards, a per-token side input, a float32 stream) at layer sizes that
 # resemble real models, beside the Tufirax design of this engine - the closest one: attention and state-space layers
@@ -1493,10 +1671,10 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the shape has (both numbers are reported)")
     ap.add_argument("--shape", default="llama-3.1-8b", choices=sorted(SHAPES), help="layer sizes of the model")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "tufirax", "vipelix", "tibepel", "tugodra", "sozudra"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "tufirax", "vipelix", "tibepel", "tugodra", "sozudra", "lefolorn"],
                     help="decode: the benchmark's one JSON line; serve: continuous batching of uneven prompts; tufirax, vipelix, tibepel, "
-                         "tugodra, sozudra: that design at real layer sizes beside the closest decoder of equal size, and its kernels alone")
-    ap.add_argument("--sizes", default="", help="tufirax, vipelix, tibepel, tugodra, sozudra: which sizes to run, with commas (default: all)")
+                         "tugodra, sozudra, lefolorn: that design at real layer sizes beside the closest decoder of equal size, and its kernels alone")
+    ap.add_argument("--sizes", default="", help="tufirax, vipelix, tibepel, tugodra, sozudra, lefolorn: which sizes to run, with commas (default: all)")
     ap.add_argument("--requests", type=int, default=64, help="serve: number of requests")
     ap.add_argument("--output-len", type=int, default=256, help="serve: tokens generated per request")
     ap.add_argument("--budget", type=int, default=2048, help="serve: tokens per step")
@@ -1524,6 +1702,8 @@ def main():
         run_tugodra(args)
     elif args.workload == "sozudra":
         run_sozudra(args)
+    elif args.workload == "lefolorn":
+        run_lefolorn(args)
     elif args.workload == "serve":
         run_serve(args)
     else:

@@ -18,6 +18,7 @@
 //
 // All arithmetic is float; storage is float or bfloat16 per argument.  Any sizes.
 #include "common.cuh"
+#include <initializer_list>
 
 __device__ __forceinline__ float lt_load(const void* p, int dtype, size_t i) {
     return dtype == RV_DTYPE_F32 ? ((const float*)p)[i] : __bfloat162float(((const __nv_bfloat16*)p)[i]);
@@ -69,30 +70,21 @@ latent_queries_kernel(const void* __restrict__ q, int in_dtype, const int* __res
     lt_queries(q, in_dtype, (size_t)t * nh * (dq + dr), t, cs, sn, half, halves, q_plain, q_row, out_dtype, nh, dq, dr, R);
 }
 
-// One block per token.  Rq > 0: the row starts with a low-rank row of the queries instead of the queries (low_out [T, Rq]).
+// One block per token.
 __global__ void __launch_bounds__(256)
 latent_prepare_kernel(const void* __restrict__ proj, int in_dtype, int row_stride, const void* __restrict__ c_gamma, int gamma_dtype,
                       const int* __restrict__ positions, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                       int rot, int table_rows, const int* __restrict__ slot_mapping, void* __restrict__ cache,
                       void* __restrict__ q_plain, void* __restrict__ q_row, int out_dtype, float* __restrict__ gate_out,
-                      int nh, int dq, int dr, int R, float eps, int write_kv, int halves, int Rq, const void* __restrict__ q_gamma,
-                      int q_gamma_dtype, void* __restrict__ low_out) {
+                      int nh, int dq, int dr, int R, float eps, int write_kv, int halves) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
     __shared__ float scratch[33];
     const int t = blockIdx.x;
     const size_t row = (size_t)t * row_stride;
-    const int qw = Rq > 0 ? Rq : nh * (dq + dr), D = R + dr;
+    const int qw = nh * (dq + dr), D = R + dr;
     const size_t c0 = row + qw;
     float ss = 0.f;
-    if (Rq > 0) {
-        for (int i = threadIdx.x; i < Rq; i += blockDim.x) { const float v = lt_load(proj, in_dtype, row + i); ss = fmaf(v, v, ss); }
-        ss = rv_block_sum(ss, scratch);
-        const float rq = 1.0f / sqrtf(ss / (float)Rq + eps);
-        for (int i = threadIdx.x; i < Rq; i += blockDim.x)
-            lt_store(low_out, out_dtype, (size_t)t * Rq + i, lt_load(proj, in_dtype, row + i) * rq * rv_load_param(q_gamma, q_gamma_dtype, i));
-        ss = 0.f;
-    }
     for (int i = threadIdx.x; i < R; i += blockDim.x) { const float v = lt_load(proj, in_dtype, c0 + i); ss = fmaf(v, v, ss); }
     ss = rv_block_sum(ss, scratch);
     const float rc = 1.0f / sqrtf(ss / (float)R + eps);
@@ -121,7 +113,7 @@ latent_prepare_kernel(const void* __restrict__ proj, int in_dtype, int row_strid
             }
         }
     }
-    if (q_plain) lt_queries(proj, in_dtype, row, t, cs, sn, half, halves, q_plain, q_row, out_dtype, nh, dq, dr, R);
+    lt_queries(proj, in_dtype, row, t, cs, sn, half, halves, q_plain, q_row, out_dtype, nh, dq, dr, R);
     if (gate_out)
         for (int h = threadIdx.x; h < nh; h += blockDim.x) {
             const float g = lt_load(proj, in_dtype, row + qw + D + h);
@@ -141,8 +133,157 @@ RV_EXPORT int rv_latent_prepare(const void* proj, int in_dtype, int row_stride, 
     if (!cos_t || !sin_t) rot = 0;
     RV_LAUNCH_ST = rv_launch(latent_prepare_kernel, dim3(n_tokens), dim3(256), 0, stream, proj, in_dtype, row_stride, c_gamma,
                              gamma_dtype, positions, cos_t, sin_t, rot, table_rows, slot_mapping, cache, q_plain, q_row, out_dtype,
-                             gate_out, nh, dq, dr, R, eps, write_kv, halves, 0, (const void*)nullptr, 0, (void*)nullptr);
+                             gate_out, nh, dq, dr, R, eps, write_kv, halves);
     return rv_launch_status();
+}
+
+// One block per token.  The row is read once, into shared memory; both statistics come from one reduction.
+__global__ void __launch_bounds__(256)
+latent_down_kernel(const void* __restrict__ proj, int in_dtype, int row_stride, const void* __restrict__ q_gamma, int q_gamma_dtype,
+                   const void* __restrict__ c_gamma, int gamma_dtype, const int* __restrict__ positions, const float* __restrict__ cos_t,
+                   const float* __restrict__ sin_t, int rot, int table_rows, const int* __restrict__ slot_mapping, void* __restrict__ cache,
+                   void* __restrict__ low_out, int out_dtype, float* __restrict__ gate_out, int nh, int Rq, int dr, int R, float eps,
+                   int write_kv, int halves) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    extern __shared__ float ld_row[];                               // [Rq + R + dr]
+    __shared__ float part[2][8];
+    const int t = blockIdx.x, n = Rq + R + dr, D = R + dr, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const size_t row = (size_t)t * row_stride;
+    const int slot = write_kv ? slot_mapping[t] : -1;
+    int pos = positions[t];
+    if (pos < 0) pos = 0;
+    if (pos >= table_rows) pos = table_rows - 1;                    // the host refuses such positions; never read outside
+    const int half = rot >> 1;
+    const float* cs = cos_t ? cos_t + (size_t)pos * half : nullptr;
+    const float* sn = sin_t ? sin_t + (size_t)pos * half : nullptr;
+    float sq = 0.f, sc = 0.f;
+    for (int i = threadIdx.x; i < n; i += 256) {
+        const float v = lt_load(proj, in_dtype, row + i);
+        ld_row[i] = v;
+        if (i < Rq) sq = fmaf(v, v, sq);
+        else if (i < Rq + R) sc = fmaf(v, v, sc);
+    }
+    sq = rv_warp_sum(sq);
+    sc = rv_warp_sum(sc);
+    if (lane == 0) { part[0][warp] = sq; part[1][warp] = sc; }
+    __syncthreads();
+    sq = sc = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) { sq += part[0][w]; sc += part[1][w]; }
+    const float rq = 1.0f / sqrtf(sq / (float)Rq + eps), rc = 1.0f / sqrtf(sc / (float)R + eps);
+    const float* rr = ld_row + Rq + R;                              // the shared rotated key part
+    for (int i = threadIdx.x; i < (slot >= 0 ? n : Rq); i += 256) {
+        if (i < Rq) {
+            lt_store(low_out, out_dtype, (size_t)t * Rq + i, ld_row[i] * rq * rv_load_param(q_gamma, q_gamma_dtype, i));
+            continue;
+        }
+        const int k = i - Rq;                                       // element of the cached row
+        float v;
+        if (k < R) {
+            v = ld_row[i] * rc * rv_load_param(c_gamma, gamma_dtype, k);
+        } else {
+            const int e = k - R;
+            v = rr[e];
+            if (e < rot) {
+                const int p = halves ? (e < half ? e : e - half) : e >> 1;
+                const bool first = halves ? e < half : !(e & 1);
+                const float other = rr[halves ? (first ? e + half : e - half) : e ^ 1];
+                v = first ? v * cs[p] - other * sn[p] : v * cs[p] + other * sn[p];
+            }
+        }
+        lt_store(cache, out_dtype, (size_t)slot * D + k, v);
+    }
+    if (gate_out)
+        for (int h = threadIdx.x; h < nh; h += 256)
+            gate_out[(size_t)t * nh + h] = 1.0f / (1.0f + expf(-lt_load(proj, in_dtype, row + n + h)));
+}
+
+__device__ __forceinline__ float4 lt_load4(const void* p, int dtype, size_t i) {          // four neighbours, i a multiple of 4
+    if (dtype == RV_DTYPE_F32) return *reinterpret_cast<const float4*>((const float*)p + i);
+    const uint2 u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+__device__ __forceinline__ void lt_store4(void* p, int dtype, size_t i, float4 v) {
+    if (dtype == RV_DTYPE_F32) {
+        *reinterpret_cast<float4*>((float*)p + i) = v;
+    } else {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        uint2 pk;
+        pk.x = *reinterpret_cast<uint32_t*>(&lo); pk.y = *reinterpret_cast<uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>((__nv_bfloat16*)p + i) = pk;
+    }
+}
+
+// The same for sizes in multiples of 4 and pairs of neighbours, without gate logits: four neighbouring elements a thread and step in
+// registers, their weights (the rotated part: cosines and sines) asked for at the same time.  NJ: steps (n <= 1024 NJ).
+template <int NJ>
+__global__ void __launch_bounds__(256)
+latent_down_vec_kernel(const float* __restrict__ proj, int row_stride, const void* __restrict__ q_gamma, int q_gamma_dtype,
+                       const void* __restrict__ c_gamma, int gamma_dtype, const int* __restrict__ positions, const float* __restrict__ cos_t,
+                       const float* __restrict__ sin_t, int rot, int table_rows, const int* __restrict__ slot_mapping, void* __restrict__ cache,
+                       void* __restrict__ low_out, int out_dtype, int Rq, int dr, int R, float eps, int write_kv) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    __shared__ float part[2][8];
+    const int t = blockIdx.x, n = Rq + R + dr, D = R + dr, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const size_t row = (size_t)t * row_stride;
+    const int slot = write_kv ? slot_mapping[t] : -1;
+    float4 v[NJ], g[NJ];
+    float sq = 0.f, sc = 0.f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        const int i = (threadIdx.x + 256 * j) * 4;
+        g[j] = make_float4(1.f, 0.f, 1.f, 0.f);                     // cos, sin, cos, sin of a pair that does not turn
+        if (i >= n) continue;
+        v[j] = *reinterpret_cast<const float4*>(proj + row + i);
+        if (i < Rq) {
+            g[j] = lt_load4(q_gamma, q_gamma_dtype, i);
+        } else if (i < Rq + R) {
+            g[j] = lt_load4(c_gamma, gamma_dtype, i - Rq);
+        } else {
+            const int e = i - Rq - R;
+            int pos = positions[t];
+            if (pos < 0) pos = 0;
+            if (pos >= table_rows) pos = table_rows - 1;            // the host refuses such positions; never read outside
+            const size_t tab = (size_t)pos * (rot >> 1) + (e >> 1);
+            if (e < rot) { g[j].x = cos_t[tab]; g[j].y = sin_t[tab]; }
+            if (e + 2 < rot) { g[j].z = cos_t[tab + 1]; g[j].w = sin_t[tab + 1]; }
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        const int i = (threadIdx.x + 256 * j) * 4;
+        if (i >= n) continue;
+        const float s = v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+        if (i < Rq) sq += s;
+        else if (i < Rq + R) sc += s;
+    }
+    sq = rv_warp_sum(sq);
+    sc = rv_warp_sum(sc);
+    if (lane == 0) { part[0][warp] = sq; part[1][warp] = sc; }
+    __syncthreads();
+    sq = sc = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) { sq += part[0][w]; sc += part[1][w]; }
+    const float rq = 1.0f / sqrtf(sq / (float)Rq + eps), rc = 1.0f / sqrtf(sc / (float)R + eps);
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        const int i = (threadIdx.x + 256 * j) * 4;
+        if (i >= n || (i >= Rq && slot < 0)) continue;
+        const float4 x = v[j], w = g[j];
+        if (i < Rq + R) {
+            const float r = i < Rq ? rq : rc;
+            const float4 y = make_float4(x.x * r * w.x, x.y * r * w.y, x.z * r * w.z, x.w * r * w.w);
+            if (i < Rq) lt_store4(low_out, out_dtype, (size_t)t * Rq + i, y);
+            else lt_store4(cache, out_dtype, (size_t)slot * D + (i - Rq), y);
+        } else {
+            lt_store4(cache, out_dtype, (size_t)slot * D + (i - Rq),
+                      make_float4(x.x * w.x - x.y * w.y, x.y * w.x + x.x * w.y, x.z * w.z - x.w * w.w, x.w * w.z + x.z * w.w));
+        }
+    }
 }
 
 // gate_out null: no gate logits in the row (nh is then of no use).
@@ -156,10 +297,68 @@ RV_EXPORT int rv_latent_down(const void* proj, int in_dtype, int row_stride, con
     if ((in_dtype | gamma_dtype | q_gamma_dtype | out_dtype) & ~1) return RV_ERR_BAD_DTYPE;
     if (n_tokens == 0) return RV_OK;
     if (!cos_t || !sin_t) rot = 0;
-    RV_LAUNCH_ST = rv_launch(latent_prepare_kernel, dim3(n_tokens), dim3(256), 0, stream, proj, in_dtype, row_stride, c_gamma,
-                             gamma_dtype, positions, cos_t, sin_t, rot, table_rows, slot_mapping, cache, (void*)nullptr, (void*)nullptr,
-                             out_dtype, gate_out, nh, 0, dr, R, eps, write_kv, halves, Rq, q_gamma, q_gamma_dtype, low_out);
+    uintptr_t bits = 0;
+    for (const void* p : {proj, q_gamma, c_gamma, (const void*)cache, (const void*)low_out}) bits |= reinterpret_cast<uintptr_t>(p);
+    if (in_dtype == RV_DTYPE_F32 && !halves && !gate_out && Rq % 4 == 0 && R % 4 == 0 && dr % 4 == 0 && row_stride % 4 == 0 && bits % 16 == 0 &&
+        Rq + R + dr <= 4096) {
+        const int steps = (Rq + R + dr + 1023) / 1024;
+        auto vec = steps <= 1 ? latent_down_vec_kernel<1> : (steps <= 2 ? latent_down_vec_kernel<2> : latent_down_vec_kernel<4>);
+        RV_LAUNCH_ST = rv_launch(vec, dim3(n_tokens), dim3(256), 0, stream, (const float*)proj, row_stride, q_gamma, q_gamma_dtype, c_gamma,
+                                 gamma_dtype, positions, cos_t, sin_t, rot, table_rows, slot_mapping, cache, low_out, out_dtype, Rq, dr, R,
+                                 eps, write_kv);
+        return rv_launch_status();
+    }
+    const size_t smem = (size_t)(Rq + R + dr) * sizeof(float);
+    if (smem > 48 * 1024 - 256) return RV_ERR_UNSUPPORTED;
+    RV_LAUNCH_ST = rv_launch(latent_down_kernel, dim3(n_tokens), dim3(256), smem, stream, proj, in_dtype, row_stride, q_gamma, q_gamma_dtype,
+                             c_gamma, gamma_dtype, positions, cos_t, sin_t, rot, table_rows, slot_mapping, cache, low_out, out_dtype, gate_out,
+                             nh, Rq, dr, R, eps, write_kv, halves);
     return rv_launch_status();
+}
+
+// bfloat16 or float rows in multiples of 4 elements, pairs of neighbours: a thread takes four neighbouring elements of a head
+__global__ void __launch_bounds__(256)
+latent_queries_vec_kernel(const float* __restrict__ q, const int* __restrict__ positions, const float* __restrict__ cos_t,
+                          const float* __restrict__ sin_t, int rot, int table_rows, void* __restrict__ q_plain, void* __restrict__ q_row,
+                          int out_dtype, int nh, int dq, int dr, int R, size_t total) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    const int per_head = (dq + dr) / 4, per_token = nh * per_head, D = R + dr;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = i / per_token;
+        const int in_token = (int)(i - t * per_token), h = in_token / per_head, e = (in_token - h * per_head) * 4;
+        float4 v = reinterpret_cast<const float4*>(q)[i];
+        void* base = q_plain;
+        size_t dst = (t * nh + h) * (size_t)dq + e;
+        if (e >= dq) {
+            const int k = e - dq;
+            base = q_row;
+            dst = (t * nh + h) * (size_t)D + R + k;
+            if (k < rot) {
+                int pos = positions[t];
+                if (pos < 0) pos = 0;
+                if (pos >= table_rows) pos = table_rows - 1;      // the host refuses such positions; never read outside
+                const size_t tab = (size_t)pos * (rot >> 1) + (k >> 1);
+                const float c0 = cos_t[tab], s0 = sin_t[tab];
+                const float x = v.x, y = v.z;
+                v.x = x * c0 - v.y * s0;
+                v.y = v.y * c0 + x * s0;
+                if (k + 2 < rot) {
+                    const float c1 = cos_t[tab + 1], s1 = sin_t[tab + 1];
+                    v.z = y * c1 - v.w * s1;
+                    v.w = v.w * c1 + y * s1;
+                }
+            }
+        }
+        if (out_dtype == RV_DTYPE_F32) {
+            *reinterpret_cast<float4*>((float*)base + dst) = v;
+        } else {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+            uint2 pk;
+            pk.x = *reinterpret_cast<uint32_t*>(&lo); pk.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>((__nv_bfloat16*)base + dst) = pk;
+        }
+    }
 }
 
 RV_EXPORT int rv_latent_queries(const void* q, int in_dtype, const int* positions, const float* cos_t, const float* sin_t, int rot,
@@ -170,6 +369,13 @@ RV_EXPORT int rv_latent_queries(const void* q, int in_dtype, const int* position
     if ((in_dtype | out_dtype) & ~1) return RV_ERR_BAD_DTYPE;
     if (n_tokens == 0) return RV_OK;
     if (!cos_t || !sin_t) { cos_t = sin_t = nullptr; rot = 0; }
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(q_plain) | reinterpret_cast<uintptr_t>(q_row);
+    if (in_dtype == RV_DTYPE_F32 && !halves && dq % 4 == 0 && dr % 4 == 0 && R % 4 == 0 && bits % 16 == 0) {
+        const size_t total = (size_t)n_tokens * nh * ((dq + dr) / 4), want = (total + 255) / 256;
+        RV_LAUNCH_ST = rv_launch(latent_queries_vec_kernel, dim3((unsigned)(want < 148 * 32 ? want : 148 * 32)), dim3(256), 0, stream,
+                                 (const float*)q, positions, cos_t, sin_t, rot, table_rows, q_plain, q_row, out_dtype, nh, dq, dr, R, total);
+        return rv_launch_status();
+    }
     RV_LAUNCH_ST = rv_launch(latent_queries_kernel, dim3(n_tokens), dim3(256), 0, stream, q, in_dtype, positions, cos_t, sin_t, rot,
                              table_rows, halves, q_plain, q_row, out_dtype, nh, dq, dr, R);
     return rv_launch_status();

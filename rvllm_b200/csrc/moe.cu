@@ -342,6 +342,65 @@ __global__ void moe_combine_kernel(const float* __restrict__ ys, const int* __re
     }
 }
 
+// The same for widths in multiples of 4: a block per token, its rows and weights in shared memory, four columns a thread and four
+// rows in flight; the sums in the same order.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(const float* __restrict__ ys, const int* __restrict__ row_of, const float* add, TO* out, int top, int width,
+                       float weight, const float* __restrict__ weights, const float* __restrict__ add_scale,
+                       const __nv_bfloat16* __restrict__ identity_x, const int* __restrict__ chosen, int experts) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    extern __shared__ float mc_smem[];                    // weights [top], rows [top] (-1: nothing, -2: the token itself)
+    int* rows = reinterpret_cast<int*>(mc_smem + top);
+    const size_t t = blockIdx.x;
+    for (int k = threadIdx.x; k < top; k += blockDim.x) {
+        const int r = row_of[t * top + k];
+        rows[k] = r >= 0 ? r : (identity_x && chosen[t * top + k] >= experts ? -2 : -1);
+        mc_smem[k] = weights ? weights[t * top + k] : 1.f;
+    }
+    __syncthreads();
+    const float scale = add && add_scale ? add_scale[t] : 1.f;
+    for (int q = threadIdx.x; q < width / 4; q += blockDim.x) {
+        const size_t at = t * width + 4 * (size_t)q;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f), s = a;
+        if (add) a = *reinterpret_cast<const float4*>(add + at);
+        for (int k0 = 0; k0 < top; k0 += 4) {
+            float4 y[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int r = k0 + j < top ? rows[k0 + j] : -1;
+                if (r >= 0) {
+                    y[j] = *reinterpret_cast<const float4*>(ys + (size_t)r * width + 4 * (size_t)q);
+                } else if (r == -2) {
+                    const uint2 u = *reinterpret_cast<const uint2*>(identity_x + at);
+                    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+                    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+                    y[j] = make_float4(lo.x, lo.y, hi.x, hi.y);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                if (k0 + j < top && rows[k0 + j] != -1) {
+                    const float w = mc_smem[k0 + j];
+                    s.x = fmaf(w, y[j].x, s.x); s.y = fmaf(w, y[j].y, s.y);
+                    s.z = fmaf(w, y[j].z, s.z); s.w = fmaf(w, y[j].w, s.w);
+                }
+            }
+        }
+        s.x = fmaf(scale, a.x, s.x * weight); s.y = fmaf(scale, a.y, s.y * weight);
+        s.z = fmaf(scale, a.z, s.z * weight); s.w = fmaf(scale, a.w, s.w * weight);
+        if constexpr (sizeof(TO) == 4) {
+            *reinterpret_cast<float4*>(out + at) = s;
+        } else {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(s.x, s.y), hi = __floats2bfloat162_rn(s.z, s.w);
+            uint2 pk;
+            pk.x = *reinterpret_cast<uint32_t*>(&lo); pk.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(out + at) = pk;
+        }
+    }
+}
+
 RV_EXPORT int rv_moe_route(const int* chosen, int pairs, int top, int experts, int block, int max_rows, int ranks, int max_units,
                            int* row_of, int* src_of, int* tile_group, int* tile_rows, int nt_a, int* order_a, int nt_b, int* order_b,
                            cudaStream_t stream) {
@@ -370,6 +429,19 @@ RV_EXPORT int rv_moe_combine(const float* ys, const int* row_of, const float* ad
     if (identity_x && (!chosen || experts <= 0)) return RV_ERR_BAD_SIZE;
     if (tokens < 0 || top <= 0 || width <= 0) return RV_ERR_BAD_SIZE;
     if (tokens == 0) return RV_OK;
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(ys) | reinterpret_cast<uintptr_t>(add) | reinterpret_cast<uintptr_t>(out) |
+                           reinterpret_cast<uintptr_t>(identity_x);
+    if (width % 4 == 0 && bits % 16 == 0 && top <= 4096) {
+        const size_t smem = (size_t)top * 8;
+        const int threads = width >= 1024 ? 256 : 128;
+        if (out_f32)
+            RV_LAUNCH_ST = rv_launch(moe_combine_vec_kernel<float>, dim3(tokens), dim3(threads), smem, stream, ys, row_of, add, (float*)out, top,
+                                     width, weight, weights, add_scale, (const __nv_bfloat16*)identity_x, chosen, experts);
+        else
+            RV_LAUNCH_ST = rv_launch(moe_combine_vec_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), smem, stream, ys, row_of, add,
+                                     (__nv_bfloat16*)out, top, width, weight, weights, add_scale, (const __nv_bfloat16*)identity_x, chosen, experts);
+        return rv_launch_status();
+    }
     const size_t total = (size_t)tokens * width;
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     if (out_f32)

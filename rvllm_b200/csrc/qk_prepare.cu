@@ -24,6 +24,7 @@
 //
 // All arithmetic is float; the results are rounded once, when they are stored (float or bfloat16).
 #include "common.cuh"
+#include <initializer_list>
 
 #define QP_WARPS 8
 #define QP_MAX_DIM 1024
@@ -31,6 +32,39 @@
 __device__ __forceinline__ void qp_store(void* p, int dtype, size_t i, float v) {
     if (dtype == RV_DTYPE_F32) ((float*)p)[i] = v;
     else ((__nv_bfloat16*)p)[i] = __float2bfloat16_rn(v);
+}
+
+// V neighbouring elements per thread and access: 4 (8 or 16 bytes) where sizes and pointers allow, else 1.
+template <int V>
+__device__ __forceinline__ void qp_load_vec(const void* p, int dtype, size_t i, float (&v)[V]) {
+    if constexpr (V == 4) {
+        if (dtype == RV_DTYPE_F32) {
+            const float4 f = *reinterpret_cast<const float4*>((const float*)p + i);
+            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+        } else {
+            const uint2 u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
+            const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+            const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+            v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+        }
+    } else {
+        v[0] = dtype == RV_DTYPE_F32 ? ((const float*)p)[i] : __bfloat162float(((const __nv_bfloat16*)p)[i]);
+    }
+}
+template <int V>
+__device__ __forceinline__ void qp_store_vec(void* p, int dtype, size_t i, const float (&v)[V]) {
+    if constexpr (V == 4) {
+        if (dtype == RV_DTYPE_F32) {
+            *reinterpret_cast<float4*>((float*)p + i) = make_float4(v[0], v[1], v[2], v[3]);
+        } else {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+            uint2 u;
+            u.x = *reinterpret_cast<uint32_t*>(&lo); u.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>((__nv_bfloat16*)p + i) = u;
+        }
+    } else {
+        qp_store(p, dtype, i, v[0]);
+    }
 }
 
 struct QkPrepareArgs {
@@ -155,6 +189,99 @@ qk_prepare_kernel(const QkPrepareArgs a) {
     }
 }
 
+// The same for one map per head whose pairs, if any, are neighbours, with sizes in multiples of 4: a warp per (token, head of q, k
+// or v), a lane holds four neighbouring elements per step (pairs never leave a lane), nothing passes through shared memory.  NJ:
+// steps (P <= 128 NJ).  Item `items` of a token is its gate logits.
+template <int NJ>
+__global__ void __launch_bounds__(QP_WARPS * 32)
+qk_prepare_vec_kernel(const QkPrepareArgs a, int items, int per_token, size_t total) {
+    rv_pdl_launch_dependents();
+    rv_pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const size_t w = (size_t)blockIdx.x * QP_WARPS + (threadIdx.x >> 5);
+    if (w >= total) return;
+    const size_t t = w / per_token;
+    const int item = (int)(w - t * per_token);
+    const size_t row = t * a.row_stride;
+    if (item >= items) {
+        const size_t g0 = row + (size_t)a.nh * a.d + (a.write_kv ? (size_t)a.nkv * (a.d + a.vd) : 0);
+        for (int h = lane; h < a.nh; h += 32) a.gate_out[t * a.nh + h] = 1.0f / (1.0f + expf(-a.proj[g0 + h]));
+        return;
+    }
+    const int kind = item < a.nh ? 0 : (item < a.nh + a.nkv ? 1 : 2);               // q, k, v
+    const int index = kind == 0 ? item : (kind == 1 ? item - a.nh : item - a.nh - a.nkv);
+    const int n = kind == 2 ? a.vd : a.d;
+    const size_t col = kind == 2 ? (size_t)(a.nh + a.nkv) * a.d + (size_t)index * a.vd : (size_t)item * a.d;
+    int pos = a.positions[t];
+    if (pos < 0) pos = 0;
+    const int slot = kind == 0 ? 0 : a.slot_mapping[t];
+    const float* cos_t = kind == 2 ? a.vcos_t : a.cos_t;
+    const float* sin_t = kind == 2 ? a.vsin_t : a.sin_t;
+    const int rot = cos_t ? (kind == 2 ? a.vd : a.rot) : 0, rows = kind == 2 ? a.v_table_rows : a.table_rows;
+    const size_t tab = (size_t)(pos < rows ? pos : rows - 1) * (rot >> 1);          // the host refuses such positions; never read outside
+    const float* gamma = kind == 0 ? a.q_gamma : (kind == 1 ? a.k_gamma : nullptr);
+    float v[NJ][4];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        const int e = (lane + 32 * j) * 4;
+        v[j][0] = v[j][1] = v[j][2] = v[j][3] = 0.f;
+        if (e < n) {
+            qp_load_vec<4>(a.proj, RV_DTYPE_F32, row + col + e, v[j]);
+            if (a.bias) {
+                float b[4];
+                qp_load_vec<4>(a.bias, RV_DTYPE_F32, col + e, b);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) v[j][i] += b[i];
+            }
+            if (kind == 2) {
+                const size_t at = (t * a.nkv + index) * a.vd + e;
+                if (a.keep_v) qp_store_vec<4>(a.keep_v, RV_DTYPE_F32, at, v[j]);
+                if (a.mix_v) {
+                    float f[4];
+                    qp_load_vec<4>(a.mix_v, RV_DTYPE_F32, at, f);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) v[j][i] = (1.0f - a.lambda) * v[j][i] + a.lambda * f[i];
+                }
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ss = fmaf(v[j][i], v[j][i], ss);                // (a turn leaves the sum as it is)
+    }
+    if (slot < 0) return;
+    float r = 1.f;
+    if (kind != 2 && (gamma || a.unit)) r = 1.0f / sqrtf(rv_warp_sum(ss) / (float)n + a.eps);
+    float post = 1.f;                                                               // behind the norm's weight
+    if (kind == 0 && a.temp_every > 0) post = 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1));
+    void* dst_base = kind == 0 ? a.q_out : a.cache;
+    const size_t page = (size_t)(slot / a.page_size), off = (size_t)(slot % a.page_size);
+    const size_t dst = kind == 0 ? (t * a.nh + index) * a.P
+                                 : (((page * 2 + (kind == 2 ? 1 : 0)) * a.nkv + index) * a.page_size + off) * a.P;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        const int e = (lane + 32 * j) * 4;
+        if (e >= a.P) continue;
+        if (e < n) {
+            float g[4] = {1.f, 1.f, 1.f, 1.f};
+            if (gamma) qp_load_vec<4>(gamma, RV_DTYPE_F32, e, g);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v[j][i] = v[j][i] * r * g[i];
+#pragma unroll
+            for (int i = 0; i < 4; i += 2) {
+                if (e + i < rot) {
+                    const float c = cos_t[tab + ((e + i) >> 1)], s = sin_t[tab + ((e + i) >> 1)];
+                    const float x = v[j][i], y = v[j][i + 1];
+                    v[j][i] = x * c - y * s;
+                    v[j][i + 1] = y * c + x * s;
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v[j][i] *= post;
+        }
+        qp_store_vec<4>(dst_base, a.out_dtype, dst + e, v[j]);
+    }
+}
+
 // q_gamma and k_gamma go together and exclude `unit`; keep_v and mix_v are float [n_tokens, nkv * vd].
 RV_EXPORT int rv_qk_prepare_ex(const float* proj, int row_stride, const float* bias, const int* positions, const float* cos_t,
                                const float* sin_t, int rot, int table_rows, int halves, const float* vcos_t, const float* vsin_t,
@@ -179,6 +306,19 @@ RV_EXPORT int rv_qk_prepare_ex(const float* proj, int row_stride, const float* b
     const QkPrepareArgs a = {proj, row_stride, bias, positions, cos_t, sin_t, rot, table_rows, halves, vcos_t, vsin_t, v_table_rows,
                              slot_mapping, cache, q_out, out_dtype, gate_out, nh, nkv, d, vd, P, maps, page_size, eps, unit, write_kv,
                              q_gamma, k_gamma, temp_coef, temp_every, keep_v, mix_v, lambda};
+    uintptr_t bits = 0;
+    for (const void* p : {(const void*)proj, (const void*)bias, (const void*)cache, (const void*)q_out, (const void*)q_gamma, (const void*)k_gamma,
+                          (const void*)keep_v, (const void*)mix_v})
+        bits |= reinterpret_cast<uintptr_t>(p);
+    if (maps == 1 && (!halves || (rot == 0 && !vcos_t)) && d % 4 == 0 && vd % 4 == 0 && P % 4 == 0 && row_stride % 4 == 0 && bits % 16 == 0) {
+        const int items = nh + (write_kv ? 2 * nkv : 0), per_token = items + (gate_out ? 1 : 0);
+        const size_t total = (size_t)n_tokens * per_token, blocks = (total + QP_WARPS - 1) / QP_WARPS;
+        if (blocks <= 0x7fffffffULL) {
+            auto vec = P <= 128 ? qk_prepare_vec_kernel<1> : (P <= 256 ? qk_prepare_vec_kernel<2> : qk_prepare_vec_kernel<8>);
+            RV_LAUNCH_ST = rv_launch(vec, dim3((unsigned)blocks), dim3(QP_WARPS * 32), 0, stream, a, items, per_token, total);
+            return rv_launch_status();
+        }
+    }
     auto kernel = P <= 32 ? qk_prepare_kernel<1> : (P <= 64 ? qk_prepare_kernel<2> : (P <= 128 ? qk_prepare_kernel<4>
                 : (P <= 256 ? qk_prepare_kernel<8> : qk_prepare_kernel<32>)));
     RV_LAUNCH_ST = rv_launch(kernel, dim3(n_tokens), dim3(QP_WARPS * 32), 0, stream, a);
@@ -196,39 +336,6 @@ RV_EXPORT int rv_qk_prepare(const float* proj, int row_stride, const float* bias
 }
 
 // ------------------------------------------------------------------ after the attention kernels
-// V neighbouring elements per thread and access: 4 (8 or 16 bytes) where sizes and pointers allow, else 1.
-template <int V>
-__device__ __forceinline__ void qp_load_vec(const void* p, int dtype, size_t i, float (&v)[V]) {
-    if constexpr (V == 4) {
-        if (dtype == RV_DTYPE_F32) {
-            const float4 f = *reinterpret_cast<const float4*>((const float*)p + i);
-            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-        } else {
-            const uint2 u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
-            const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
-            const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-            v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
-        }
-    } else {
-        v[0] = dtype == RV_DTYPE_F32 ? ((const float*)p)[i] : __bfloat162float(((const __nv_bfloat16*)p)[i]);
-    }
-}
-template <int V>
-__device__ __forceinline__ void qp_store_vec(void* p, int dtype, size_t i, const float (&v)[V]) {
-    if constexpr (V == 4) {
-        if (dtype == RV_DTYPE_F32) {
-            *reinterpret_cast<float4*>((float*)p + i) = make_float4(v[0], v[1], v[2], v[3]);
-        } else {
-            __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
-            uint2 u;
-            u.x = *reinterpret_cast<uint32_t*>(&lo); u.y = *reinterpret_cast<uint32_t*>(&hi);
-            *reinterpret_cast<uint2*>((__nv_bfloat16*)p + i) = u;
-        }
-    } else {
-        qp_store(p, dtype, i, v[0]);
-    }
-}
-
 // A thread takes V neighbouring pairs.  halves: pairs (m, m + vd / 2); else (2m, 2m + 1), V = 1.
 template <int V>
 __global__ void __launch_bounds__(256)

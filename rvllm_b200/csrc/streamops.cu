@@ -514,7 +514,7 @@ struct GatedArgs {
     int cols;
 };
 
-__device__ __forceinline__ float so_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float so_sigmoid(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }      // (a few units in the last place)
 __device__ __forceinline__ float4 so_load4(const void* p, int dtype, size_t i) {          // four neighbours, i a multiple of 4
     if (dtype == RV_DTYPE_F32) return *reinterpret_cast<const float4*>((const float*)p + i);
     const uint2 u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
@@ -525,7 +525,7 @@ __device__ __forceinline__ float4 so_load4(const void* p, int dtype, size_t i) {
 
 // A row per block.  NV > 0: 4 columns a thread and access, the row in registers, every 32 accesses of a warp inside one group
 // (cols / 4 / groups a multiple of 32); NV = 0: any width and groups, the row is read again for the norm.
-template <int NV>
+template <int NV, int TERMS>
 __global__ void __launch_bounds__(256)
 gated_combine_kernel(const GatedArgs a) {
     rv_pdl_launch_dependents();
@@ -539,31 +539,25 @@ gated_combine_kernel(const GatedArgs a) {
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
             const int i = threadIdx.x + j * blockDim.x;
-            if (i < quads) v[j] = reinterpret_cast<const float4*>(a.x + base)[i];
-        }
+            if (i >= quads) continue;
+            v[j] = reinterpret_cast<const float4*>(a.x + base)[i];
+            if (TERMS == 0) continue;
+            float4 y[TERMS ? TERMS : 1], g[TERMS ? TERMS : 1];           // the row's own loads first: they come from memory, the vectors from a cache
 #pragma unroll
-        for (int k = 0; k < 2; ++k) {
-            if (k >= a.terms) break;
+            for (int k = 0; k < TERMS; ++k) {
+                y[k] = reinterpret_cast<const float4*>(a.y[k] + base)[i];
+                g[k] = so_load4(a.gates, a.gates_dtype, gbase + (size_t)k * a.cols + 4 * i);
+            }
 #pragma unroll
-            for (int j = 0; j < NV; ++j) {
-                const int i = threadIdx.x + j * blockDim.x;
-                if (i >= quads) continue;
-                const float4 y = reinterpret_cast<const float4*>(a.y[k] + base)[i];
+            for (int k = 0; k < TERMS; ++k) {
                 const float4 s = reinterpret_cast<const float4*>(a.scale[k])[i];
                 const float4 b = reinterpret_cast<const float4*>(a.bias + (size_t)k * a.cols)[i];
-                const float4 g = so_load4(a.gates, a.gates_dtype, gbase + (size_t)k * a.cols + 4 * i);
-                v[j].x = fmaf(y.x * s.x, so_sigmoid(g.x + b.x), v[j].x);
-                v[j].y = fmaf(y.y * s.y, so_sigmoid(g.y + b.y), v[j].y);
-                v[j].z = fmaf(y.z * s.z, so_sigmoid(g.z + b.z), v[j].z);
-                v[j].w = fmaf(y.w * s.w, so_sigmoid(g.w + b.w), v[j].w);
+                v[j].x = fmaf(y[k].x * s.x, so_sigmoid(g[k].x + b.x), v[j].x);
+                v[j].y = fmaf(y[k].y * s.y, so_sigmoid(g[k].y + b.y), v[j].y);
+                v[j].z = fmaf(y[k].z * s.z, so_sigmoid(g[k].z + b.z), v[j].z);
+                v[j].w = fmaf(y[k].w * s.w, so_sigmoid(g[k].w + b.w), v[j].w);
             }
-        }
-        if (a.terms) {
-#pragma unroll
-            for (int j = 0; j < NV; ++j) {
-                const int i = threadIdx.x + j * blockDim.x;
-                if (i < quads) reinterpret_cast<float4*>(a.x + base)[i] = v[j];
-            }
+            reinterpret_cast<float4*>(a.x + base)[i] = v[j];
         }
         if (!a.gamma) return;
 #pragma unroll
@@ -622,6 +616,12 @@ gated_combine_kernel(const GatedArgs a) {
     }
 }
 
+template <int TERMS>
+static void (*gated_pick(int nv))(const GatedArgs) {
+    return nv <= 1 ? gated_combine_kernel<1, TERMS> : (nv <= 2 ? gated_combine_kernel<2, TERMS> : (nv <= 4 ? gated_combine_kernel<4, TERMS>
+                                                                                                          : gated_combine_kernel<8, TERMS>));
+}
+
 // y0, y1: float terms, the first null one ends them; scale0, scale1 float [cols]; gates [rows, g_stride] and bias float [terms * cols];
 // gamma null: no norm and no `out`.
 RV_EXPORT int rv_gated_combine(float* x, const float* y0, const float* scale0, const float* y1, const float* scale1, const void* gates,
@@ -642,11 +642,12 @@ RV_EXPORT int rv_gated_combine(float* x, const float* y0, const float* scale0, c
     if (gamma) bits |= reinterpret_cast<uintptr_t>(gamma) | reinterpret_cast<uintptr_t>(out);
     const int threads = cols >= 1024 ? 256 : 128;
     const int nv = (cols / 4 + threads - 1) / threads;
-    auto kernel = gated_combine_kernel<0>;
+    auto kernel = gated_combine_kernel<0, 0>;                            // (this one reads the number of terms from its arguments)
     size_t smem = (gamma ? groups : 1) * sizeof(float);
     if (cols % 4 == 0 && g_stride % 4 == 0 && bits % 16 == 0 && nv <= 8 && (!gamma || (cols / 4) % (32 * groups) == 0)) {
-        kernel = nv <= 1 ? gated_combine_kernel<1> : (nv <= 2 ? gated_combine_kernel<2> : (nv <= 4 ? gated_combine_kernel<4>
-                                                                                                : gated_combine_kernel<8>));
+        kernel = gated_pick<0>(nv);
+        if (terms == 1) kernel = gated_pick<1>(nv);
+        if (terms == 2) kernel = gated_pick<2>(nv);
         smem = (size_t)8 * (threads / 32) * sizeof(float);
     }
     RV_LAUNCH_ST = rv_launch(kernel, dim3(rows), dim3(threads), smem, stream, a);

@@ -47,6 +47,8 @@ class LatentAttention(Part):
             problems.append("sizes must be positive")
         if q_rank is not None and q_rank < 1:
             problems.append(f"the queries' latent needs at least one element, got {q_rank}")
+        if q_rank is not None and q_rank + kv_rank + rot_dim > 12000:
+            problems.append(f"the two latents and the rotated part together have at most 12,000 elements, got {q_rank} + {kv_rank} + {rot_dim}")
         if rot_dim % 2:
             problems.append(f"the rotated part must have an even size, got {rot_dim}")
         if pairs not in ("neighbours", "halves"):
