@@ -479,6 +479,15 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                         s0[e] = __float_as_uint(fmaf(__uint_as_float(s0[e]), sc, bias_far));
                         s1[e] = __float_as_uint(fmaf(__uint_as_float(s1[e]), sc, bias_far));
                     }
+                } else if (__all_sync(0xffffffffu, pos < 0 || (key0 + KV_TILE - 1 <= pos && key0 > far_from))) {
+                    // every key of the tile has an entry of its own for every row that counts (a row beyond the last reads those of a
+                    // distance that some other row of the warp has)
+                    const float* entry = bias_row + (pos < 0 ? KV_TILE - 1 : pos - key0) * G;
+#pragma unroll
+                    for (int e = 0; e < 32; ++e) {
+                        s0[e] = __float_as_uint(fmaf(__uint_as_float(s0[e]), sc, __ldg(entry - e * G)));
+                        s1[e] = __float_as_uint(fmaf(__uint_as_float(s1[e]), sc, __ldg(entry - (e + 32) * G)));
+                    }
                 } else {
 #pragma unroll
                     for (int e = 0; e < 32; ++e) {
