@@ -526,7 +526,7 @@ __device__ __forceinline__ float4 so_load4(const void* p, int dtype, size_t i) {
 // A row per block.  NV > 0: 4 columns a thread and access, the row in registers, every 32 accesses of a warp inside one group
 // (cols / 4 / groups a multiple of 32); NV = 0: any width and groups, the row is read again for the norm.
 template <int NV, int TERMS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(512)
 gated_combine_kernel(const GatedArgs a) {
     rv_pdl_launch_dependents();
     rv_pdl_wait();
@@ -640,7 +640,7 @@ RV_EXPORT int rv_gated_combine(float* x, const float* y0, const float* scale0, c
     if (terms) bits |= reinterpret_cast<uintptr_t>(y0) | reinterpret_cast<uintptr_t>(scale0) | reinterpret_cast<uintptr_t>(gates) | reinterpret_cast<uintptr_t>(bias);
     if (terms > 1) bits |= reinterpret_cast<uintptr_t>(y1) | reinterpret_cast<uintptr_t>(scale1);
     if (gamma) bits |= reinterpret_cast<uintptr_t>(gamma) | reinterpret_cast<uintptr_t>(out);
-    const int threads = cols >= 1024 ? 256 : 128;
+    const int threads = cols >= 4096 ? 512 : (cols >= 1024 ? 256 : 128);
     const int nv = (cols / 4 + threads - 1) / threads;
     auto kernel = gated_combine_kernel<0, 0>;                            // (this one reads the number of terms from its arguments)
     size_t smem = (gamma ? groups : 1) * sizeof(float);
